@@ -95,7 +95,8 @@ class ModelSpec:
     # a position encoding that adds to the embeddings before the first block (learned or
     # absolute positions); None: positions enter inside the mixers only
     embedding_position: PartSpec = None
-    # logits <- cap * tanh(logits / cap); 0: none
+    # logits <- scale * logits, then cap * tanh(logits / cap); cap 0: none
+    logit_scale: float = 1.0
     logit_softcap: float = 0.0
     # the embedding rows are multiplied by this on their way into the 32-bit stream
     embedding_scale: float = 1.0

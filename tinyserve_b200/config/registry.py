@@ -14,6 +14,7 @@ import os
 from .babadra import BabadraConfig
 from .delilorn import DelilornConfig
 from .dudatar import DudatarConfig
+from .gunulorn import GunulornConfig
 from .model_config import ConfigError, ModelConfig, Qwen3Config
 from .tarivik import TarivikConfig
 
@@ -66,3 +67,4 @@ register_architecture(DudatarConfig.architecture, DudatarConfig)
 register_architecture(DelilornConfig.architecture, DelilornConfig)
 register_architecture(TarivikConfig.architecture, TarivikConfig)
 register_architecture(BabadraConfig.architecture, BabadraConfig)
+register_architecture(GunulornConfig.architecture, GunulornConfig)

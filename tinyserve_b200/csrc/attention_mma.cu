@@ -65,6 +65,7 @@ struct MmaAttnParams {
   const float* sinks;       // [H] or null
   int chunk;                // > 0: a query at position i sees key j only if i / chunk == j / chunk (no window then)
   const float* slopes;      // [H] or null: slopes[h] * (i - j) is taken off head h's scaled score
+  TurnBack turn;            // outputs turned back by their query's position; cos null: none
   float scale_log2;
   // a soft cap c > 0 on the scaled score s, c tanh(s / c): cap2 = c log2(e) (0: none), cap_in = scale / c
   float cap2, cap_in;
@@ -384,9 +385,17 @@ __global__ void __launch_bounds__(PRE_THREADS) attn_prefill_kernel(MmaAttnParams
     const float inv = sum > 0.f ? alpha / sum : 0.f;
     bf16* dst = p.out + ((size_t)(q_begin + q0 + qi) * p.H + kvh * G + g0 + gg) * D;
 #pragma unroll
-    for (int dt = 0; dt < D / 8; ++dt)
-      *reinterpret_cast<__nv_bfloat162*>(dst + dt * 8 + 2 * t) =
-          __floats2bfloat162_rn(o[dt][2 * h] * inv, o[dt][2 * h + 1] * inv);
+    for (int dt = 0; dt < D / 8; ++dt) {
+      float a = o[dt][2 * h] * inv, b = o[dt][2 * h + 1] * inv;
+      const int m2 = dt * 4 + t;                       // the column pair
+      if (p.turn.cos && m2 < p.turn.half) {
+        const size_t at = (size_t)pos[h] * p.turn.half + m2;
+        const float cs = p.turn.cos[at], sn = p.turn.sin[at], u = a;
+        a = u * cs + b * sn;
+        b = b * cs - u * sn;
+      }
+      *reinterpret_cast<__nv_bfloat162*>(dst + dt * 8 + 2 * t) = __floats2bfloat162_rn(a, b);
+    }
   }
 }
 
@@ -737,7 +746,14 @@ __device__ __forceinline__ void attn_decode_body(const MmaAttnParams& p, const C
   }
   __syncthreads();
   const bool stores = !TMA || abort_flag_s == 0;
+  // (a turned output needs its column's mate, which is the neighbour lane's: both lanes of a pair are in or out)
+  auto finished = [&](float v, int d, unsigned lanes) {
+    if (!p.turn.cos) return v;
+    const float mate = __shfl_xor_sync(lanes, v, 1);
+    return p.turn.value(v, mate, d, qpos);
+  };
   for (int i = threadIdx.x; i < ng * D; i += THREADS) {
+    const unsigned lanes = ~0u >> (32 - min(32, ng * D - (i - lane)));        // the warp's lanes of this round
     const int r = i / D, d = i % D;
     float mx = -INFINITY;
 #pragma unroll
@@ -761,7 +777,8 @@ __device__ __forceinline__ void attn_decode_body(const MmaAttnParams& p, const C
       mx = m_new;
     }
     if (p.num_splits == 1) {
-      if (stores) p.out[((size_t)q_begin * p.H + head) * D + d] = __float2bfloat16_rn(den > 0.f ? num / den : 0.f);
+      const float y = finished(den > 0.f ? num / den : 0.f, d, lanes);
+      if (stores) p.out[((size_t)q_begin * p.H + head) * D + d] = __float2bfloat16_rn(y);
     } else if (p.cluster_merge) {
       // this thread has read its four values of (r, d); the first warp's place now holds their sum
       sm_o[r * D + d] = num;
@@ -784,9 +801,10 @@ __device__ __forceinline__ void attn_decode_body(const MmaAttnParams& p, const C
     // its share of the (head, dimension) pairs from all ranks' shared memory, in rank order.
     cluster_arrive();
     cluster_wait();
-    const int per_rank = (ng * D + p.num_splits - 1) / p.num_splits;
+    const int per_rank = ((ng * D + p.num_splits - 1) / p.num_splits + 1) & ~1;       // (whole column pairs)
     const int i_end = min(ng * D, (split + 1) * per_rank);
     for (int i = split * per_rank + threadIdx.x; i < i_end; i += THREADS) {
+      const unsigned lanes = ~0u >> (32 - min(32, i_end - (i - lane)));
       const int r = i / D, d = i % D;
       float ms[8], ls[8], os[8];
 #pragma unroll
@@ -808,7 +826,8 @@ __device__ __forceinline__ void attn_decode_body(const MmaAttnParams& p, const C
           num = fmaf(wgt, os[s], num);
           den = fmaf(wgt, ls[s], den);
         }
-      if (stores) p.out[((size_t)q_begin * p.H + kvh * G + g0 + r) * D + d] = __float2bfloat16_rn(den > 0.f ? num / den : 0.f);
+      const float y = finished(den > 0.f ? num / den : 0.f, d, lanes);
+      if (stores) p.out[((size_t)q_begin * p.H + kvh * G + g0 + r) * D + d] = __float2bfloat16_rn(y);
     }
     if (traced) timeline_mark_thread(45, split);        // merged and stored
     // no block leaves while a peer may still read its shared memory
@@ -834,7 +853,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
 // a negative token marks an unused entry of the list)
 __global__ void attention_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                          bf16* __restrict__ out, int num_splits, int H,
-                                         const int* __restrict__ tokens) {
+                                         const int* __restrict__ tokens, TurnBack turn) {
   pdl_trigger();
   pdl_wait();
   const size_t row = blockIdx.x;
@@ -846,13 +865,21 @@ __global__ void attention_combine_kernel(const float* __restrict__ part_o, const
   float den = 0.f;
   for (int s = 0; s < num_splits; ++s) den += ml[2 * s] == -INFINITY ? 0.f : exp2f(ml[2 * s] - mx) * ml[2 * s + 1];
   const float inv = den > 0.f ? 1.f / den : 0.f;
-  for (int d = threadIdx.x; d < D; d += blockDim.x) {
+  const int pos = turn.cos ? turn.positions[out_row / H] : 0;
+  for (int d0 = 0; d0 < D; d0 += blockDim.x) {       // (whole warps take every round)
+    const int d = d0 + threadIdx.x;
     float v = 0.f;
-    for (int s = 0; s < num_splits; ++s) {
-      const float w = ml[2 * s] == -INFINITY ? 0.f : exp2f(ml[2 * s] - mx);
-      v = fmaf(w, part_o[(row * num_splits + s) * D + d], v);
+    if (d < D)
+      for (int s = 0; s < num_splits; ++s) {
+        const float w = ml[2 * s] == -INFINITY ? 0.f : exp2f(ml[2 * s] - mx);
+        v = fmaf(w, part_o[(row * num_splits + s) * D + d], v);
+      }
+    v *= inv;
+    if (turn.cos) {
+      const float mate = __shfl_xor_sync(0xffffffffu, v, 1);
+      if (d < D) v = turn.value(v, mate, d, pos);
     }
-    out[out_row * D + d] = __float2bfloat16_rn(v * inv);
+    if (d < D) out[out_row * D + d] = __float2bfloat16_rn(v);
   }
 }
 
@@ -893,7 +920,9 @@ TS_EXPORT int ts_paged_attention_mma(const void* q, void* out, const void* k_cac
                                      int num_splits, float* part_o, float* part_ml,
                                      int decode_only, const int* tile_req, const int* tile_q0, int num_tiles,
                                      int tile_queries, int num_pages, int keep_first, const float* sinks,
-                                     int chunk, const float* slopes, float softcap, int v_share, cudaStream_t stream) {
+                                     int chunk, const float* slopes, float softcap, int v_share, const float* turn_cos,
+                                     const float* turn_sin, int turn_half, const int* positions, cudaStream_t stream) {
+  TS_REQUIRE(turn_cos == nullptr || (turn_sin && positions && turn_half > 0 && 2 * turn_half <= D), "paged_attention_mma: turned outputs of %d pairs in heads of %d", turn_half, D);
   TS_REQUIRE(keep_first >= 0, "paged_attention_mma: keep_first %d", keep_first);
   TS_REQUIRE(chunk >= 0 && (chunk == 0 || window <= 0), "paged_attention_mma: a chunk of %d positions (and no window beside it)", chunk);
   MmaAttnParams extra = {};
@@ -901,6 +930,7 @@ TS_EXPORT int ts_paged_attention_mma(const void* q, void* out, const void* k_cac
   extra.sinks = sinks;
   extra.chunk = chunk;
   extra.slopes = slopes;
+  extra.turn = TurnBack{turn_cos, turn_sin, turn_half, positions};
   if (softcap > 0.f) { extra.cap2 = softcap * LOG2E; extra.cap_in = scale / softcap; }
   return paged_attention_mma_impl(&extra, q, out, k_cache, v_cache, block_table, cu_q, kv_lens, num_tokens,
                                   num_requests, max_q_len, H, Hkv, page_size, max_blocks, scale, window, num_splits,
@@ -1024,7 +1054,7 @@ int paged_attention_mma_impl(const MmaAttnParams* from_qkv, const void* q, void*
     if (num_splits > 1) {
       TS_LAUNCH("attention_combine", attention_combine_kernel, (tile_req ? count : num_tokens) * H,
                 D >= 128 ? 128 : (D >= 64 ? 64 : 32), 0, stream,
-                (const float*)part_o, (const float*)part_ml, p.out, num_splits, H, tile_q0);
+                (const float*)part_o, (const float*)part_ml, p.out, num_splits, H, tile_q0, p.turn);
     }
     return 0;
   }

@@ -8,7 +8,8 @@
 // (and, with a window W > 0, j > position - W or j < keep_first: the first keys of a sequence
 // may stay visible to every query behind them); query head h reads KV head h / (H / Hkv);
 // with `sinks`, head h's softmax sum also holds exp(sinks[h]), a term without key or value;
-// keys are found through the request's block table.  Online softmax as
+// keys are found through the request's block table.  With a TurnBack every output row is turned back by
+// its query's position before it is stored (values that were turned to theirs).  Online softmax as
 // tinykernels.py:386-413, but with every product and sum in 32-bit.
 //
 // A block handles 32 rows = (query, head of one KV group) pairs, so that one pass over the
@@ -52,6 +53,7 @@ struct AttnParams {
   int chunk;                // > 0: a query at position i sees key j only if i / chunk == j / chunk (no window then)
   const float* slopes;      // [H] or null: slopes[h] * (i - j) is taken off the score of head h
   float scale;
+  TurnBack turn;            // cos null: none
   float softcap;            // > 0: the scaled score s becomes softcap * tanh(s / softcap) (before the slopes' bias)
 };
 
@@ -225,9 +227,16 @@ __global__ void __launch_bounds__(WARPS * 32) paged_attention_kernel(AttnParams 
       }
       const float inv = l[i] > 0.f ? 1.f / l[i] : 0.f;
       T* o = static_cast<T*>(p.out) + row * D;
+      const int pos = pos0 + qi;
 #pragma unroll
-      for (int c = 0; c < DC; ++c)
-        if (D % 32 == 0 || lane + 32 * c < D) o[lane + 32 * c] = from_f32<T>(acc[i][c] * inv);
+      for (int c = 0; c < DC; ++c) {
+        float v = acc[i][c] * inv;
+        if (p.turn.cos) {
+          const float mate = __shfl_xor_sync(0xffffffffu, v, 1);      // (a row is the whole warp's)
+          if (D % 32 == 0 || lane + 32 * c < D) v = p.turn.value(v, mate, lane + 32 * c, pos);
+        }
+        if (D % 32 == 0 || lane + 32 * c < D) o[lane + 32 * c] = from_f32<T>(v);
+      }
     } else {
       float* o = p.part_o + (row * p.num_splits + split) * D;
 #pragma unroll
@@ -245,7 +254,7 @@ __global__ void __launch_bounds__(WARPS * 32) paged_attention_kernel(AttnParams 
 template <typename T>
 __global__ void attention_combine_kernel(const float* __restrict__ part_o,
                                          const float* __restrict__ part_ml, T* __restrict__ out,
-                                         int num_splits, const float* __restrict__ sinks, int H) {
+                                         int num_splits, const float* __restrict__ sinks, int H, TurnBack turn) {
   pdl_trigger();
   pdl_wait();
   const size_t row = blockIdx.x;
@@ -258,13 +267,21 @@ __global__ void attention_combine_kernel(const float* __restrict__ part_o,
   for (int s = 0; s < num_splits; ++s)
     denom += (ml[2 * s] == -INFINITY) ? 0.f : expf(ml[2 * s] - m) * ml[2 * s + 1];
   const float inv = denom > 0.f ? 1.f / denom : 0.f;
-  for (int d = threadIdx.x; d < D; d += blockDim.x) {
+  const int pos = turn.cos ? turn.positions[row / H] : 0;
+  for (int d0 = 0; d0 < D; d0 += blockDim.x) {       // (whole warps take every round)
+    const int d = d0 + threadIdx.x;
     float v = 0.f;
-    for (int s = 0; s < num_splits; ++s) {
-      const float w = (ml[2 * s] == -INFINITY) ? 0.f : expf(ml[2 * s] - m);
-      v = fmaf(w, part_o[(row * num_splits + s) * D + d], v);
+    if (d < D)
+      for (int s = 0; s < num_splits; ++s) {
+        const float w = (ml[2 * s] == -INFINITY) ? 0.f : expf(ml[2 * s] - m);
+        v = fmaf(w, part_o[(row * num_splits + s) * D + d], v);
+      }
+    v *= inv;
+    if (turn.cos) {
+      const float mate = __shfl_xor_sync(0xffffffffu, v, 1);
+      if (d < D) v = turn.value(v, mate, d, pos);
     }
-    out[row * D + d] = from_f32<T>(v * inv);
+    if (d < D) out[row * D + d] = from_f32<T>(v);
   }
 }
 
@@ -284,7 +301,9 @@ TS_EXPORT int ts_paged_attention_biased(int dtype, const void* q, void* out, con
                                         int max_q_len, int H, int Hkv, int page_size, int max_blocks,
                                         float scale, int window, int num_splits, float* part_o,
                                         float* part_ml, int keep_first, const float* sinks, int chunk,
-                                        const float* slopes, float softcap, int v_share, cudaStream_t stream) {
+                                        const float* slopes, float softcap, int v_share, const float* turn_cos,
+                                        const float* turn_sin, int turn_half, const int* positions, cudaStream_t stream) {
+  TS_REQUIRE(turn_cos == nullptr || (turn_sin && positions && turn_half > 0 && 2 * turn_half <= D), "paged_attention: turned outputs of %d pairs in heads of %d", turn_half, D);
   TS_REQUIRE(num_tokens > 0 && num_requests > 0 && max_q_len > 0, "paged_attention: empty batch");
   TS_REQUIRE(v_share >= 1 && Hkv % v_share == 0, "paged_attention: %d key heads do not share values in runs of %d", Hkv, v_share);
   TS_REQUIRE(chunk >= 0 && (chunk == 0 || window <= 0), "paged_attention: a chunk of %d positions (and no window beside it)", chunk);
@@ -307,6 +326,7 @@ TS_EXPORT int ts_paged_attention_biased(int dtype, const void* q, void* out, con
   p.num_splits = num_splits; p.window = window; p.scale = scale;
   p.keep_first = keep_first; p.sinks = sinks;
   p.chunk = chunk; p.slopes = slopes; p.softcap = softcap;
+  p.turn = TurnBack{turn_cos, turn_sin, turn_half, positions};
   const long long gz = (long long)num_requests * num_splits;
   const long long gy = (long long)Hkv * p.head_tiles;
   TS_REQUIRE(gz <= 65535 && gy <= 65535, "paged_attention: grid too large (%lld requests*splits, %lld head tiles)", gz, gy);
@@ -325,9 +345,9 @@ TS_EXPORT int ts_paged_attention_biased(int dtype, const void* q, void* out, con
   if (num_splits > 1) {
     const int threads = D >= 128 ? 128 : (D >= 64 ? 64 : 32);
     if (dtype == TS_F32)
-      TS_LAUNCH("attention_combine", attention_combine_kernel<float>, num_tokens * H, threads, 0, stream, (const float*)part_o, (const float*)part_ml, (float*)out, num_splits, sinks, H);
+      TS_LAUNCH("attention_combine", attention_combine_kernel<float>, num_tokens * H, threads, 0, stream, (const float*)part_o, (const float*)part_ml, (float*)out, num_splits, sinks, H, p.turn);
     else
-      TS_LAUNCH("attention_combine", attention_combine_kernel<__nv_bfloat16>, num_tokens * H, threads, 0, stream, (const float*)part_o, (const float*)part_ml, (__nv_bfloat16*)out, num_splits, sinks, H);
+      TS_LAUNCH("attention_combine", attention_combine_kernel<__nv_bfloat16>, num_tokens * H, threads, 0, stream, (const float*)part_o, (const float*)part_ml, (__nv_bfloat16*)out, num_splits, sinks, H, p.turn);
   }
   return 0;
 }
@@ -340,7 +360,7 @@ TS_EXPORT int ts_paged_attention(int dtype, const void* q, void* out, const void
                                  float* part_ml, int keep_first, const float* sinks, cudaStream_t stream) {
   return ts_paged_attention_biased(dtype, q, out, k_cache, v_cache, block_table, cu_q, kv_lens, num_tokens, num_requests,
                                    max_q_len, H, Hkv, page_size, max_blocks, scale, window, num_splits, part_o, part_ml,
-                                   keep_first, sinks, 0, nullptr, 0.f, 1, stream);
+                                   keep_first, sinks, 0, nullptr, 0.f, 1, nullptr, nullptr, 0, nullptr, stream);
 }
 
 // ------------------------------------------------------------------ no-allocation entry point

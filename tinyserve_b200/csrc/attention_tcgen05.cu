@@ -78,6 +78,7 @@ struct TcAttnParams {
   const float* sinks;       // [H] or null: one more term exp(sinks[h]) in every softmax sum of head h
   int chunk;                // > 0: a query at position i sees key j only if i / chunk == j / chunk (no window then)
   const float* slopes;      // [H] or null: slopes[h] * (i - j) is taken off head h's scaled score
+  TurnBack turn;            // outputs turned back by their query's position; cos null: none
   float scale_log2;
   // a soft cap c > 0 on the scaled score s, c tanh(s / c): cap2 = c log2(e) (0: none), cap_in = scale / c
   float cap2, cap_in;
@@ -468,6 +469,17 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
         for (int c = 0; c < D; c += 32) {
           float v[32];
           tmem_load32(tmem_o + lane_addr + c, v);
+          if (p.turn.cos && valid && c < 2 * p.turn.half) {
+            const size_t at = (size_t)pos * p.turn.half + (c >> 1);
+#pragma unroll
+            for (int e = 0; e < 32; e += 2) {
+              if (c + e < 2 * p.turn.half) {
+                const float cs = p.turn.cos[at + e / 2], sn = p.turn.sin[at + e / 2], a = v[e], b = v[e + 1];
+                v[e] = a * cs + b * sn;
+                v[e + 1] = b * cs - a * sn;
+              }
+            }
+          }
           if (valid) {
 #pragma unroll
             for (int e = 0; e < 32; e += 8)
@@ -525,7 +537,9 @@ TS_EXPORT int ts_paged_attention_tcgen05(const void* q, void* out, const void* k
                                          int num_pages, int page_size, int max_blocks, float scale, int window,
                                          const int* tile_req, const int* tile_q0, int num_tiles,
                                          int tile_queries, int keep_first, const float* sinks, int chunk,
-                                         const float* slopes, float softcap, int v_share, cudaStream_t stream) {
+                                         const float* slopes, float softcap, int v_share, const float* turn_cos,
+                                         const float* turn_sin, int turn_half, const int* positions, cudaStream_t stream) {
+  TS_REQUIRE(turn_cos == nullptr || (turn_sin && turn_half > 0 && 2 * turn_half <= D), "paged_attention_tcgen05: turned outputs of %d pairs in heads of %d", turn_half, D);
   TS_REQUIRE(keep_first >= 0, "paged_attention_tcgen05: keep_first %d", keep_first);
   TS_REQUIRE(v_share >= 1 && Hkv % v_share == 0, "paged_attention_tcgen05: %d key heads do not share values in runs of %d", Hkv, v_share);
   TS_REQUIRE(chunk >= 0 && (chunk == 0 || window <= 0), "paged_attention_tcgen05: a chunk of %d positions (and no window beside it)", chunk);
@@ -544,6 +558,7 @@ TS_EXPORT int ts_paged_attention_tcgen05(const void* q, void* out, const void* k
   p.v_share = v_share; p.Hv = Hkv / v_share;
   p.keep_first = keep_first; p.sinks = sinks;
   p.chunk = chunk; p.slopes = slopes;
+  p.turn = TurnBack{turn_cos, turn_sin, turn_half, positions};
   p.page_shift = 0;
   while ((1 << p.page_shift) < page_size) ++p.page_shift;
   p.scale_log2 = scale * 1.4426950408889634f;

@@ -241,6 +241,22 @@ struct VecParam {
   }
 };
 
+// Attention over values that were turned to their tokens' positions: the query's output is turned back by its own
+// position, column pair (2m, 2m + 1) by -position * f_m.  cos and sin [positions, half] hold the angles of the first
+// 2 half columns; cos null: nothing turns.  `mine` is column d of a row and `mate` column d ^ 1.
+struct TurnBack {
+  const float* cos;
+  const float* sin;
+  int half;
+  const int* positions;     // [T], for the kernels that know a row by its token only
+  __device__ __forceinline__ float value(float mine, float mate, int d, int pos) const {
+    if (d >= 2 * half) return mine;
+    const size_t at = (size_t)pos * half + (d >> 1);
+    const float c = cos[at], s = sin[at];
+    return d & 1 ? mine * c - mate * s : mine * c + mate * s;
+  }
+};
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

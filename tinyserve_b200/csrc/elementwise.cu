@@ -457,6 +457,333 @@ TS_EXPORT int ts_add_rmsnorm(int dtype, const void* x, float* residual, const vo
   return ts_fail("add_rmsnorm: unknown dtype %d", dtype);
 }
 
+// ------------------------------------------------------------------ addends of two branches + RMSNorm with two weights
+// Row r of the 32-bit residual takes in what a block of two branches left: up to two tensors stored as T, the
+// partial tiles of one product, one vector for all rows and row_factor[r] times a row of another tensor (any of
+// them absent).  The sum's norm leaves with one or two weights, out_i = v * rsqrt(mean(v^2) + eps) * w_i: the
+// inputs of the two branches of the next block.  Few rows: a row over a cluster of NORM_CLUSTER blocks.
+struct BranchAddends {
+  const void* x1;            // [rows, n] or null
+  const void* x2;            // [rows, n] or null
+  PartialSrc ps;             // base null: none
+  VecParam bias;             // [n]; ptr null: none
+  const float* row_factor;   // [rows] or null
+  const void* row_src;       // [rows, n]
+};
+
+template <typename T>
+__device__ __forceinline__ float branch_addend1(const BranchAddends& a, size_t r, int c, int n) {
+  float v = 0.f;
+  if (a.ps.base) v += a.ps.load1((int)r, c);
+  if (a.x1) v += to_f32<T>(static_cast<const T*>(a.x1)[r * n + c]);
+  if (a.x2) v += to_f32<T>(static_cast<const T*>(a.x2)[r * n + c]);
+  if (a.bias.ptr) v += a.bias[c];
+  if (a.row_factor) v = fmaf(a.row_factor[r], to_f32<T>(static_cast<const T*>(a.row_src)[r * n + c]), v);
+  return v;
+}
+
+template <typename T>
+__global__ void branch_norm_kernel(BranchAddends a, float* __restrict__ residual, VecParam w1, VecParam w2, float eps,
+                                   T* __restrict__ out1, T* __restrict__ out2, const int* __restrict__ rows, int n,
+                                   int write_residual) {
+  __shared__ float scratch[33];
+  pdl_trigger();
+  pdl_wait();
+  const size_t i = blockIdx.x, r = rows ? (size_t)rows[i] : i;
+  float* rr = residual + r * n;
+  float acc = 0.f;
+  for (int c = threadIdx.x; c < n; c += blockDim.x) {
+    const float v = rr[c] + branch_addend1<T>(a, r, c, n);
+    acc += v * v;
+  }
+  const float rstd = rsqrtf(block_sum(acc, scratch) / (float)n + eps);
+  for (int c = threadIdx.x; c < n; c += blockDim.x) {
+    const float v = rr[c] + branch_addend1<T>(a, r, c, n);
+    if (write_residual) rr[c] = v;
+    out1[i * n + c] = from_f32<T>(v * rstd * w1[c]);
+    if (out2) out2[i * n + c] = from_f32<T>(v * rstd * w2[c]);
+  }
+}
+
+__device__ __forceinline__ void quad_param(const VecParam& w, int c, float (&v)[4]) {
+  if (w.is_f32) Quad<float>::load(static_cast<const float*>(w.ptr) + c, v);
+  else Quad<__nv_bfloat16>::load(static_cast<const __nv_bfloat16*>(w.ptr) + c, v);
+}
+
+template <typename T, int ITEMS, bool CLUSTER, int MAX_THREADS = 1024, int MIN_BLOCKS = 1>
+__global__ void __launch_bounds__(MAX_THREADS, MIN_BLOCKS)
+branch_norm_vec_kernel(BranchAddends a, float* __restrict__ residual, VecParam w1, VecParam w2, float eps,
+                       T* __restrict__ out1, T* __restrict__ out2, const int* __restrict__ rows, int n,
+                       int quads_per_block, int write_residual) {
+  __shared__ float scratch[33];
+  __shared__ float cluster_part;
+  pdl_trigger();
+  const int base = CLUSTER ? (int)cluster_rank() * quads_per_block : 0;
+  pdl_wait();
+  const size_t i = CLUSTER ? blockIdx.y : blockIdx.x;
+  const size_t r = rows ? (size_t)rows[i] : i;
+  const float factor = a.row_factor ? a.row_factor[r] : 0.f;
+  float v[ITEMS][4];
+  float acc = 0.f;
+#pragma unroll
+  for (int it = 0; it < ITEMS; ++it) {
+    const int q = threadIdx.x + it * blockDim.x, c = (base + q) * 4;
+    if (q >= quads_per_block || c >= n) continue;
+    Quad<float>::load(residual + r * n + c, v[it]);
+    float add[4] = {0.f, 0.f, 0.f, 0.f}, t[4];
+    if (!CLUSTER && a.ps.base) a.ps.load4((int)r, c, add);
+    if (CLUSTER && a.ps.base) {
+      // all loads of a batch are issued before the first is used; the sum runs in split order
+      for (int s0 = 0; s0 < a.ps.splits; s0 += PARTIAL_BATCH) {
+        float4 part[PARTIAL_BATCH];
+#pragma unroll
+        for (int s = 0; s < PARTIAL_BATCH; ++s)
+          if (s0 + s < a.ps.splits) part[s] = __ldcg(reinterpret_cast<const float4*>(a.ps.base + a.ps.offset(s0 + s, (int)r, c)));
+#pragma unroll
+        for (int s = 0; s < PARTIAL_BATCH; ++s)
+          if (s0 + s < a.ps.splits) { add[0] += part[s].x; add[1] += part[s].y; add[2] += part[s].z; add[3] += part[s].w; }
+      }
+    }
+    if (a.x1) {
+      Quad<T>::load(static_cast<const T*>(a.x1) + r * n + c, t);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) add[e] += t[e];
+    }
+    if (a.x2) {
+      Quad<T>::load(static_cast<const T*>(a.x2) + r * n + c, t);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) add[e] += t[e];
+    }
+    if (a.bias.ptr) {
+      quad_param(a.bias, c, t);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) add[e] += t[e];
+    }
+    if (a.row_factor) {
+      Quad<T>::load(static_cast<const T*>(a.row_src) + r * n + c, t);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) add[e] = fmaf(factor, t[e], add[e]);
+    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      v[it][e] += add[e];
+      acc += v[it][e] * v[it][e];
+    }
+  }
+  float total = block_sum(acc, scratch);
+  if (CLUSTER) {
+    if (threadIdx.x == 0) cluster_part = total;
+    cluster_arrive();
+    cluster_wait();
+    total = 0.f;
+#pragma unroll
+    for (int k = 0; k < NORM_CLUSTER; ++k) total += cluster_load_f32(&cluster_part, k);
+    cluster_arrive();        // this block has read its peers; it may not leave before they have read it
+  }
+  const float rstd = rsqrtf(total / (float)n + eps);
+#pragma unroll
+  for (int it = 0; it < ITEMS; ++it) {
+    const int q = threadIdx.x + it * blockDim.x, c = (base + q) * 4;
+    if (q >= quads_per_block || c >= n) continue;
+    if (write_residual) Quad<float>::store(residual + r * n + c, v[it]);
+    float wv[4], o[4];
+    quad_param(w1, c, wv);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) o[e] = v[it][e] * rstd * wv[e];
+    Quad<T>::store(out1 + i * n + c, o);
+    if (out2) {
+      quad_param(w2, c, wv);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) o[e] = v[it][e] * rstd * wv[e];
+      Quad<T>::store(out2 + i * n + c, o);
+    }
+  }
+  if (CLUSTER) cluster_wait();
+}
+
+template <typename T>
+int launch_branch_norm(const BranchAddends& a, float* residual, VecParam w1, VecParam w2, float eps, void* out1, void* out2,
+                       const int* rows, int num_out, int n, int write_residual, cudaStream_t stream) {
+  const bool aligned = n % 4 == 0 && ((uintptr_t)a.x1 | (uintptr_t)a.x2 | (uintptr_t)a.row_src | (uintptr_t)a.bias.ptr |
+                                      (uintptr_t)residual | (uintptr_t)out1 | (uintptr_t)out2 | (uintptr_t)w1.ptr |
+                                      (uintptr_t)w2.ptr) % 16 == 0;
+  T *o1 = (T*)out1, *o2 = (T*)out2;
+  const int quads = n / 4;
+  if (aligned && num_out <= 64 && n >= 1024 && n <= NORM_CLUSTER * 4 * 256) {
+    const int per = (quads + NORM_CLUSTER - 1) / NORM_CLUSTER;
+    cudaError_t e = ts_launch_cluster(branch_norm_vec_kernel<T, 1, true, 256>, dim3(NORM_CLUSTER, num_out), dim3((per + 31) / 32 * 32), 0,
+                                      stream, dim3(NORM_CLUSTER), a, residual, w1, w2, eps, o1, o2, rows, n, per, write_residual);
+    if (e != cudaSuccess) return ts_fail("branch_norm: %s", cudaGetErrorString(e));
+    return 0;
+  }
+  if (aligned && n <= 4 * 4 * 1024) {
+    int items = quads <= 1024 ? 1 : (quads <= 2048 ? 2 : 4);
+    if (num_out >= 512 && quads >= 256) items = quads <= 512 ? 2 : 4;
+    const int threads = ((quads + items - 1) / items + 31) / 32 * 32;
+#define TS_BRANCH_NORM(...) TS_LAUNCH("branch_norm", (branch_norm_vec_kernel<T, __VA_ARGS__>), num_out, threads, 0, stream, a, residual, w1, w2, eps, o1, o2, rows, n, quads, write_residual)
+    if (items == 1) TS_BRANCH_NORM(1, false);
+    else if (items == 2 && threads <= 256) TS_BRANCH_NORM(2, false, 256, 5);
+    else if (items == 2) TS_BRANCH_NORM(2, false);
+    else if (threads <= 256) TS_BRANCH_NORM(4, false, 256, 4);
+    else TS_BRANCH_NORM(4, false);
+#undef TS_BRANCH_NORM
+    return 0;
+  }
+  const int threads = n >= 2048 ? 512 : (n >= 512 ? 256 : 128);
+  TS_LAUNCH("branch_norm", branch_norm_kernel<T>, num_out, threads, 0, stream, a, residual, w1, w2, eps, o1, o2, rows, n, write_residual);
+  return 0;
+}
+
+// residual [., n] (float, in place with write_residual) += x1 + x2 + partial tiles + bias + row_factor * row_src; out1 (and
+// out2, with w2) [num_out, n] the sum's RMS norm times w1 (w2).  With `rows` output row i is row rows[i].
+TS_EXPORT int ts_branch_norm(int dtype, const void* x1, const void* x2, const float* partials, int splits, int n_tiles, int t_tiles,
+                             int tile_t, const void* bias, int bias_is_f32, const float* row_factor, const void* row_src,
+                             float* residual, const void* w1, const void* w2, int w_is_f32, float eps, void* out1, void* out2,
+                             const int* rows, int num_out, int n, int write_residual, cudaStream_t stream) {
+  TS_REQUIRE(num_out > 0 && n > 0 && residual && w1 && out1 && (w2 == nullptr) == (out2 == nullptr), "branch_norm: empty input");
+  TS_REQUIRE(partials == nullptr || (splits > 0 && n_tiles * 128 >= n && tile_t > 0), "branch_norm: partial tiles do not fit the row length");
+  TS_REQUIRE(row_factor == nullptr || row_src, "branch_norm: row factors without their rows");
+  const BranchAddends a{x1, x2, PartialSrc{partials, splits, n_tiles, t_tiles, tile_t}, VecParam{bias, bias_is_f32}, row_factor, row_src};
+  const VecParam v1{w1, w_is_f32}, v2{w2, w_is_f32};
+  if (dtype == TS_F32)
+    return launch_branch_norm<float>(a, residual, v1, v2, eps, out1, out2, rows, num_out, n, write_residual, stream);
+  if (dtype == TS_BF16)
+    return launch_branch_norm<__nv_bfloat16>(a, residual, v1, v2, eps, out1, out2, rows, num_out, n, write_residual, stream);
+  return ts_fail("branch_norm: unknown dtype %d", dtype);
+}
+
+// out [rows, n] = x + bias + row_factor[r] * row_src[r] (x null: nothing), stored as T
+template <typename T>
+__global__ void add_rows_kernel(BranchAddends a, T* __restrict__ out, int n) {
+  pdl_trigger();
+  pdl_wait();
+  const size_t r = blockIdx.x;
+  for (int c = threadIdx.x; c < n; c += blockDim.x) out[r * n + c] = from_f32<T>(branch_addend1<T>(a, r, c, n));
+}
+
+TS_EXPORT int ts_add_rows(int dtype, const void* x, const float* row_factor, const void* row_src, void* out, int num_rows, int n,
+                          cudaStream_t stream) {
+  TS_REQUIRE(num_rows > 0 && n > 0 && row_factor && row_src && out, "add_rows: empty input");
+  const BranchAddends a{x, nullptr, PartialSrc{nullptr, 0, 0, 0, 1}, VecParam{nullptr, 0}, row_factor, row_src};
+  if (dtype == TS_F32) TS_LAUNCH("add_rows", add_rows_kernel<float>, num_rows, 256, 0, stream, a, (float*)out, n);
+  else if (dtype == TS_BF16) TS_LAUNCH("add_rows", add_rows_kernel<__nv_bfloat16>, num_rows, 256, 0, stream, a, (__nv_bfloat16*)out, n);
+  else return ts_fail("add_rows: unknown dtype %d", dtype);
+  return 0;
+}
+
+// ------------------------------------------------------------------ a polynomial of normed powers
+// out = c0 N(z) + c1 N(z^2) + c2 N(z^3) + c3, element by element, N(y) = y / sqrt(mean(y^2) + eps) over the row.
+// One pass adds up z^2, z^4 and z^6; a thread keeps its first HOLD chunks of 16 bytes between the passes and reads
+// any further ones twice.
+template <typename T> struct Chunk16 { static constexpr int N = 16 / sizeof(T); };
+template <typename T>
+__device__ __forceinline__ void chunk16_floats(const uint4& raw, float (&v)[Chunk16<T>::N]) {
+  const T* e = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+  for (int i = 0; i < Chunk16<T>::N; ++i) v[i] = to_f32<T>(e[i]);
+}
+
+struct PolyFactors { float r1, r2, r3, e; };
+__device__ __forceinline__ PolyFactors poly_factors(float s2, float s4, float s6, const VecParam& coef, int n, float eps) {
+  const float inv = 1.f / (float)n;
+  return PolyFactors{coef[0] * rsqrtf(s2 * inv + eps), coef[1] * rsqrtf(s4 * inv + eps), coef[2] * rsqrtf(s6 * inv + eps), coef[3]};
+}
+__device__ __forceinline__ float poly_value(float z, const PolyFactors& f) {
+  return fmaf(z, fmaf(z, fmaf(z, f.r3, f.r2), f.r1), f.e);
+}
+__device__ __forceinline__ void poly_sums(float z, float& s2, float& s4, float& s6) {
+  const float q = z * z, q2 = q * q;
+  s2 += q;
+  s4 += q2;
+  s6 = fmaf(q2, q, s6);
+}
+
+template <typename T, int HOLD>      // HOLD 0: any row length and alignment, element by element
+__global__ void poly_norm_kernel(const T* __restrict__ z, T* __restrict__ out, VecParam coef, float eps, int n) {
+  __shared__ float scratch[33];
+  pdl_trigger();
+  pdl_wait();
+  const T* row = z + (size_t)blockIdx.x * n;
+  T* dst = out + (size_t)blockIdx.x * n;
+  float s2 = 0.f, s4 = 0.f, s6 = 0.f;
+  if constexpr (HOLD == 0) {
+    for (int c = threadIdx.x; c < n; c += blockDim.x) poly_sums(to_f32<T>(row[c]), s2, s4, s6);
+    s2 = block_sum(s2, scratch); s4 = block_sum(s4, scratch); s6 = block_sum(s6, scratch);
+    const PolyFactors f = poly_factors(s2, s4, s6, coef, n, eps);
+    for (int c = threadIdx.x; c < n; c += blockDim.x) dst[c] = from_f32<T>(poly_value(to_f32<T>(row[c]), f));
+  } else {
+    constexpr int N = Chunk16<T>::N;
+    const int chunks = n / N;
+    uint4 held[HOLD];
+#pragma unroll
+    for (int k = 0; k < HOLD; ++k) {
+      const int c = threadIdx.x + k * blockDim.x;
+      if (c < chunks) held[k] = reinterpret_cast<const uint4*>(row)[c];
+    }
+#pragma unroll
+    for (int k = 0; k < HOLD; ++k) {
+      const int c = threadIdx.x + k * blockDim.x;
+      if (c >= chunks) break;
+      float v[N];
+      chunk16_floats<T>(held[k], v);
+#pragma unroll
+      for (int e = 0; e < N; ++e) poly_sums(v[e], s2, s4, s6);
+    }
+    for (int c = threadIdx.x + HOLD * blockDim.x; c < chunks; c += blockDim.x) {
+      float v[N];
+      chunk16_floats<T>(reinterpret_cast<const uint4*>(row)[c], v);
+#pragma unroll
+      for (int e = 0; e < N; ++e) poly_sums(v[e], s2, s4, s6);
+    }
+    s2 = block_sum(s2, scratch); s4 = block_sum(s4, scratch); s6 = block_sum(s6, scratch);
+    const PolyFactors f = poly_factors(s2, s4, s6, coef, n, eps);
+    auto put = [&](int c, const uint4& raw) {
+      float v[N];
+      chunk16_floats<T>(raw, v);
+      uint4 o;
+      T* oe = reinterpret_cast<T*>(&o);
+#pragma unroll
+      for (int e = 0; e < N; ++e) oe[e] = from_f32<T>(poly_value(v[e], f));
+      reinterpret_cast<uint4*>(dst)[c] = o;
+    };
+#pragma unroll
+    for (int k = 0; k < HOLD; ++k) {
+      const int c = threadIdx.x + k * blockDim.x;
+      if (c < chunks) put(c, held[k]);
+    }
+    for (int c = threadIdx.x + HOLD * blockDim.x; c < chunks; c += blockDim.x) put(c, reinterpret_cast<const uint4*>(row)[c]);
+  }
+}
+
+template <typename T>
+int launch_poly_norm(const void* z, void* out, VecParam coef, float eps, int rows, int n, cudaStream_t stream) {
+  const T* zp = (const T*)z;
+  T* op = (T*)out;
+  const int N = 16 / (int)sizeof(T);
+  if (n % N == 0 && ((uintptr_t)z | (uintptr_t)out) % 16 == 0) {
+    const int chunks = n / N;
+    // few rows: the shortest chain; many rows: more rows in flight per SM
+    const int threads = rows < 512 ? (chunks >= 1024 ? 1024 : (chunks + 31) / 32 * 32) : (chunks >= 512 ? 256 : (chunks >= 128 ? 128 : 32));
+    const int hold = (chunks + threads - 1) / threads;
+    if (hold <= 1) TS_LAUNCH("poly_norm", (poly_norm_kernel<T, 1>), rows, threads, 0, stream, zp, op, coef, eps, n);
+    else if (hold <= 2) TS_LAUNCH("poly_norm", (poly_norm_kernel<T, 2>), rows, threads, 0, stream, zp, op, coef, eps, n);
+    else if (hold <= 4) TS_LAUNCH("poly_norm", (poly_norm_kernel<T, 4>), rows, threads, 0, stream, zp, op, coef, eps, n);
+    else TS_LAUNCH("poly_norm", (poly_norm_kernel<T, 6>), rows, threads, 0, stream, zp, op, coef, eps, n);
+    return 0;
+  }
+  TS_LAUNCH("poly_norm", (poly_norm_kernel<T, 0>), rows, n >= 2048 ? 512 : 128, 0, stream, zp, op, coef, eps, n);
+  return 0;
+}
+
+// z, out [rows, n]; coef four numbers
+TS_EXPORT int ts_poly_norm(int dtype, const void* z, void* out, const void* coef, int coef_is_f32, float eps, int rows, int n,
+                           cudaStream_t stream) {
+  TS_REQUIRE(rows > 0 && n > 0 && z && out && coef, "poly_norm: empty input");
+  if (dtype == TS_F32) return launch_poly_norm<float>(z, out, VecParam{coef, coef_is_f32}, eps, rows, n, stream);
+  if (dtype == TS_BF16) return launch_poly_norm<__nv_bfloat16>(z, out, VecParam{coef, coef_is_f32}, eps, rows, n, stream);
+  return ts_fail("poly_norm: unknown dtype %d", dtype);
+}
+
 // plain RMSNorm of rows stored as T
 template <typename T>
 __global__ void rmsnorm_kernel(const T* __restrict__ x, VecParam w, float eps, T* __restrict__ out,
@@ -1218,19 +1545,19 @@ TS_EXPORT int ts_sum2(int dtype, const void* a, const void* b, void* out, long l
 }
 
 // ------------------------------------------------------------------ soft cap of logits
-// x <- cap * tanh(x / cap), in place, 32-bit
-__global__ void softcap_kernel(float* __restrict__ x, size_t count, float cap) {
+// x <- cap * tanh(scale * x / cap), in place, 32-bit; cap 0: x <- scale * x
+__global__ void softcap_kernel(float* __restrict__ x, size_t count, float cap, float scale) {
   pdl_trigger();
   pdl_wait();
-  const float inv = 1.f / cap;
+  const float in = cap > 0.f ? scale / cap : scale;
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < count; i += (size_t)gridDim.x * blockDim.x)
-    x[i] = cap * tanhf(x[i] * inv);
+    x[i] = cap > 0.f ? cap * tanhf(x[i] * in) : x[i] * in;
 }
 
-TS_EXPORT int ts_softcap(float* x, long long count, float cap, cudaStream_t stream) {
-  TS_REQUIRE(count > 0 && cap > 0.f, "softcap: empty input or a cap that is not positive");
+TS_EXPORT int ts_softcap(float* x, long long count, float cap, float scale, cudaStream_t stream) {
+  TS_REQUIRE(count > 0 && cap >= 0.f, "softcap: empty input or a negative cap");
   const int blocks = (int)((count + 255) / 256 < 8192 ? (count + 255) / 256 : 8192);
-  TS_LAUNCH("softcap", softcap_kernel, blocks, 256, 0, stream, x, (size_t)count, cap);
+  TS_LAUNCH("softcap", softcap_kernel, blocks, 256, 0, stream, x, (size_t)count, cap, scale);
   return 0;
 }
 
@@ -1398,7 +1725,8 @@ __global__ void rope_unit_kvwrite_kernel(const T* __restrict__ q, long long ldq,
                                          const int* __restrict__ positions, RopeArgs rope, int unit_norm, float eps,
                                          int H, int G, int dim, int vdim, int D, T* __restrict__ k_cache,
                                          T* __restrict__ v_cache, const int* __restrict__ slot_mapping, int page_size,
-                                         int heads_total, VecParam qw, VecParam kw, float pre_eps, int maps) {
+                                         int heads_total, VecParam qw, VecParam kw, float pre_eps, int maps,
+                                         const float* __restrict__ vcos, const float* __restrict__ vsin) {
   pdl_trigger();
   pdl_wait();
   const int warps = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -1426,6 +1754,18 @@ __global__ void rope_unit_kvwrite_kernel(const T* __restrict__ q, long long ldq,
         // the value cache holds G / maps heads: the maps of a key/value head read the same one
         src = v + (size_t)t * ldv + (size_t)g * vdim;
         dst = v_cache + ((page * (G / maps) + g) * page_size + in_page) * D;
+        if (vcos) {      // pair (2m, 2m + 1) of the value turns to the token's position
+          const size_t at = (size_t)positions[t] * (vdim >> 1);
+          for (int i = lane; i < D; i += 32) {
+            float y = 0.f;
+            if (i < vdim) {
+              const float a = to_f32<T>(src[i]), b = to_f32<T>(src[i ^ 1]), c = vcos[at + (i >> 1)], s = vsin[at + (i >> 1)];
+              y = i & 1 ? a * c + b * s : a * c - b * s;
+            }
+            dst[i] = from_f32<T>(y);
+          }
+          continue;
+        }
         for (int i = lane; i < D; i += 32) dst[i] = i < vdim ? src[i] : from_f32<T>(0.f);
         continue;
       }
@@ -1467,12 +1807,108 @@ __global__ void rope_unit_kvwrite_kernel(const T* __restrict__ q, long long ldq,
   }
 }
 
+// The same for neighbouring pairs without norms and maps, sizes in multiples of 8: a thread turns eight columns of a
+// stored head (four pairs), 16 bytes of bfloat16 or two times 16 bytes of float in and out.
+template <typename T>
+__device__ __forceinline__ void load8(const T* p, float (&v)[8]);
+template <>
+__device__ __forceinline__ void load8<float>(const float* p, float (&v)[8]) {
+  const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+template <>
+__device__ __forceinline__ void load8<__nv_bfloat16>(const __nv_bfloat16* p, float (&v)[8]) {
+  chunk16_floats<__nv_bfloat16>(*reinterpret_cast<const uint4*>(p), v);
+}
+template <typename T>
+__device__ __forceinline__ void store8(T* p, const float (&v)[8]);
+template <>
+__device__ __forceinline__ void store8<float>(float* p, const float (&v)[8]) {
+  reinterpret_cast<float4*>(p)[0] = make_float4(v[0], v[1], v[2], v[3]);
+  reinterpret_cast<float4*>(p)[1] = make_float4(v[4], v[5], v[6], v[7]);
+}
+template <>
+__device__ __forceinline__ void store8<__nv_bfloat16>(__nv_bfloat16* p, const float (&v)[8]) {
+  uint4 raw;
+  __nv_bfloat162* e = reinterpret_cast<__nv_bfloat162*>(&raw);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) e[i] = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+  *reinterpret_cast<uint4*>(p) = raw;
+}
+__device__ __forceinline__ void turn_pairs8(float (&v)[8], const float* __restrict__ cos, const float* __restrict__ sin, size_t at) {
+  const float4 c = *reinterpret_cast<const float4*>(cos + at), s = *reinterpret_cast<const float4*>(sin + at);
+  const float cs[4] = {c.x, c.y, c.z, c.w}, sn[4] = {s.x, s.y, s.z, s.w};
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const float a = v[2 * i], b = v[2 * i + 1];
+    v[2 * i] = a * cs[i] - b * sn[i];
+    v[2 * i + 1] = b * cs[i] + a * sn[i];
+  }
+}
+
+template <typename T>
+__global__ void rope_pairs_kvwrite_kernel(const T* __restrict__ q, long long ldq, const T* __restrict__ k, long long ldk,
+                                          const T* __restrict__ v, long long ldv, T* __restrict__ q_out,
+                                          const int* __restrict__ positions, const float* __restrict__ cos,
+                                          const float* __restrict__ sin, int R, const float* __restrict__ vcos,
+                                          const float* __restrict__ vsin, int H, int G, int dim, int vdim, int D,
+                                          T* __restrict__ k_cache, T* __restrict__ v_cache, const int* __restrict__ slot_mapping,
+                                          int page_size, int heads_total) {
+  pdl_trigger();
+  pdl_wait();
+  const int t = blockIdx.x, per = D >> 3;
+  for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < heads_total * per; i += gridDim.y * blockDim.x) {
+    const int head = i / per, c0 = (i % per) * 8;
+    const bool is_q = head < H, is_v = head >= H + G;
+    const int g = is_q ? head : (is_v ? head - H - G : head - H);
+    const T* src = is_q ? q + (size_t)t * ldq + (size_t)g * dim : (is_v ? v + (size_t)t * ldv + (size_t)g * vdim : k + (size_t)t * ldk + (size_t)g * dim);
+    T* dst;
+    if (is_q) {
+      dst = q_out + ((size_t)t * H + g) * D;
+    } else {
+      const int slot = slot_mapping[t];
+      if (slot < 0) continue;
+      const size_t page = slot / page_size, in_page = slot % page_size;
+      dst = (is_v ? v_cache : k_cache) + ((page * G + g) * page_size + in_page) * D;
+    }
+    float x[8];
+    if (c0 < (is_v ? vdim : dim)) {
+      load8<T>(src + c0, x);
+      if (is_v) {
+        if (vcos) turn_pairs8(x, vcos, vsin, (size_t)positions[t] * (vdim >> 1) + (c0 >> 1));
+      } else if (c0 < R) {
+        turn_pairs8(x, cos, sin, (size_t)positions[t] * (R >> 1) + (c0 >> 1));
+      }
+    } else {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x[e] = 0.f;
+    }
+    store8<T>(dst + c0, x);
+  }
+}
+
+template <typename T>
+int launch_rope_pairs(const void* q, long long ldq, const void* k, long long ldk, const void* v, long long ldv, void* q_out,
+                      const int* positions, const float* cos, const float* sin, int R, const float* vcos, const float* vsin,
+                      int num_tokens, int H, int G, int dim, int vdim, int D, void* k_cache, void* v_cache, const int* slot_mapping,
+                      int page_size, int heads_total, cudaStream_t stream) {
+  const int items = heads_total * (D / 8), threads = 128;
+  const int tiles = (items + threads - 1) / threads;
+  const dim3 grid(num_tokens, num_tokens >= 256 ? (tiles < 2 ? tiles : 2) : tiles);
+  TS_LAUNCH("rope_pairs_kvwrite", rope_pairs_kvwrite_kernel<T>, grid, threads, 0, stream, (const T*)q, ldq, (const T*)k, ldk,
+            (const T*)v, ldv, (T*)q_out, positions, cos, sin, R, vcos, vsin, H, G, dim, vdim, D, (T*)k_cache, (T*)v_cache,
+            slot_mapping, page_size, heads_total);
+  return 0;
+}
+
+// vcos / vsin [positions, vdim / 2] (or null): every value head is turned to its token's position, in pairs (2m, 2m + 1)
 TS_EXPORT int ts_rope_unit_kvwrite(int dtype, const void* q, long long ldq, const void* k, long long ldk, const void* v,
                                    long long ldv, void* q_out, const int* positions, const float* cos, const float* sin,
                                    int rotary_dim, int interleaved, int unit_norm, float eps, int num_tokens, int H, int G,
                                    int dim, int vdim, int D, void* k_cache, void* v_cache, const int* slot_mapping,
                                    int page_size, const void* q_weight, const void* k_weight, int weights_are_f32,
-                                   float pre_eps, int maps, cudaStream_t stream) {
+                                   float pre_eps, int maps, const float* vcos, const float* vsin, cudaStream_t stream) {
+  TS_REQUIRE((vcos == nullptr) == (vsin == nullptr) && (vcos == nullptr || vdim % 2 == 0), "rope_unit_kvwrite: a value head of %d columns does not turn in pairs", vdim);
   TS_REQUIRE(num_tokens > 0 && H > 0 && G > 0 && dim > 0 && vdim > 0 && D >= dim && D >= vdim,
              "rope_unit_kvwrite: sizes do not fit (dim %d, vdim %d, stored head size %d)", dim, vdim, D);
   TS_REQUIRE(maps >= 1 && H % maps == 0 && G % maps == 0 && H % G == 0, "rope_unit_kvwrite: %d maps do not divide %d and %d heads", maps, H, G);
@@ -1482,6 +1918,17 @@ TS_EXPORT int ts_rope_unit_kvwrite(int dtype, const void* q, long long ldq, cons
   TS_REQUIRE(rotary_dim == 0 || (cos && sin), "rope_unit_kvwrite: rotary without tables");
   TS_REQUIRE(slot_mapping == nullptr || (k_cache && v_cache && page_size > 0), "rope_unit_kvwrite: cache write without a cache");
   const int heads_total = slot_mapping ? H + G + G / maps : H;
+  if ((interleaved || rotary_dim == 0) && !unit_norm && !q_weight && maps == 1 && ((dim | vdim | D | rotary_dim) & 7) == 0 &&
+      ((ldq | ldk | ldv) & 7) == 0 &&
+      (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)q_out | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)cos | (uintptr_t)sin |
+        (uintptr_t)vcos | (uintptr_t)vsin) & 15) == 0) {
+    if (dtype == TS_F32)
+      return launch_rope_pairs<float>(q, ldq, k, ldk, v, ldv, q_out, positions, cos, sin, rotary_dim, vcos, vsin, num_tokens, H, G, dim,
+                                      vdim, D, k_cache, v_cache, slot_mapping, page_size, heads_total, stream);
+    if (dtype == TS_BF16)
+      return launch_rope_pairs<__nv_bfloat16>(q, ldq, k, ldk, v, ldv, q_out, positions, cos, sin, rotary_dim, vcos, vsin, num_tokens, H,
+                                              G, dim, vdim, D, k_cache, v_cache, slot_mapping, page_size, heads_total, stream);
+  }
   const int warps = num_tokens >= 256 ? 8 : 4;
   dim3 grid(num_tokens, num_tokens >= 256 ? 1 : (heads_total + warps - 1) / warps);
   RopeArgs rope{cos, sin, rotary_dim, interleaved};
@@ -1489,12 +1936,12 @@ TS_EXPORT int ts_rope_unit_kvwrite(int dtype, const void* q, long long ldq, cons
   if (dtype == TS_F32)
     TS_LAUNCH("rope_unit_kvwrite", rope_unit_kvwrite_kernel<float>, grid, warps * 32, 0, stream, (const float*)q, ldq,
               (const float*)k, ldk, (const float*)v, ldv, (float*)q_out, positions, rope, unit_norm, eps, H, G, dim, vdim, D,
-              (float*)k_cache, (float*)v_cache, slot_mapping, page_size, heads_total, qw, kw, pre_eps, maps);
+              (float*)k_cache, (float*)v_cache, slot_mapping, page_size, heads_total, qw, kw, pre_eps, maps, vcos, vsin);
   else if (dtype == TS_BF16)
     TS_LAUNCH("rope_unit_kvwrite", rope_unit_kvwrite_kernel<__nv_bfloat16>, grid, warps * 32, 0, stream,
               (const __nv_bfloat16*)q, ldq, (const __nv_bfloat16*)k, ldk, (const __nv_bfloat16*)v, ldv,
               (__nv_bfloat16*)q_out, positions, rope, unit_norm, eps, H, G, dim, vdim, D, (__nv_bfloat16*)k_cache,
-              (__nv_bfloat16*)v_cache, slot_mapping, page_size, heads_total, qw, kw, pre_eps, maps);
+              (__nv_bfloat16*)v_cache, slot_mapping, page_size, heads_total, qw, kw, pre_eps, maps, vcos, vsin);
   else
     return ts_fail("rope_unit_kvwrite: unknown dtype %d", dtype);
   return 0;

@@ -17,6 +17,11 @@
 // last adds the partials in split order (so the sum is the same every run) and writes the
 // output.  Nobody waits for anybody.  Counters return to zero for the next call.
 //
+// Two forms take several operand pairs (a block of two branches, whose input products and whose output products
+// would otherwise be two launches each).  Beside: products of different x, W with one K, every row tile belongs
+// to one of them and writes to its output.  Chained: out = x1 W1^T + x2 W2^T, the K slices of the second pair
+// follow those of the first into the same accumulators.
+//
 // Every mbarrier wait is bounded: if a wait runs out, the block raises the library's error flag
 // (ts_gemm_tcgen05_error), lets its copies land, frees its tensor memory and returns.
 // tinyserve leaves these products to cuBLAS (serve.py:847, 883, 916, 919, 1263).
@@ -36,6 +41,17 @@ constexpr int BK = 64;               // K elements of a stage: 128 bytes, one sw
 constexpr int ISSUERS = BK / 16;     // issuing threads: one per K step of a stage, each with its own accumulator
 constexpr int THREADS = 32 * (1 + ISSUERS);      // warp 0 loads, warps 1..4 issue, warps 0..3 do the epilogue
 constexpr int W_STAGE_BYTES = TILE_N * BK * 2;
+
+// one of the products of the beside form
+struct GemmSegment {
+  void* out;            // [M, ldc]
+  int N, ldc, out_f32;
+  int tile0;            // its first row tile in the grid
+  VecParam bias;        // [N] or null
+};
+constexpr int MAX_SEGMENTS = 3;
+struct Maps1 { CUtensorMap w[1], x[1]; };
+struct Maps3 { CUtensorMap w[MAX_SEGMENTS], x[MAX_SEGMENTS]; };
 
 struct GemmParams {
   void* out;            // [M, ldc] bfloat16 or float
@@ -62,6 +78,16 @@ struct GemmParams {
   float gated_limit;    // the bound of a bounded activation (gated_value)
   VecParam bias;        // [N] added to every token's result (plain output only); ptr null: none
   VecParam res_scale;   // residual form: [N] factors on the result before it joins the residual; ptr null: none
+  // the forms with several operand pairs (Maps3)
+  int segments;         // beside: how many products; 0: chained
+  GemmSegment seg[MAX_SEGMENTS];
+  int kb_first, kb_all; // chained: K slices of the first pair, of both
+  // chained residual form: `bias` joins the result, and so does row_factor[m] * row_src[m, n] (null: not);
+  // hprime2 (or null) = bfloat16(residual * norm_w2) for the other branch of the next block
+  const float* row_factor;
+  const bf16* row_src;
+  VecParam norm_w2;
+  bf16* hprime2;
 };
 constexpr int SUMSQ_STRIDE = 16;     // tokens of the residual form (one token tile of 16)
 
@@ -96,10 +122,11 @@ template <int TILE_T> struct Cfg {
   static constexpr size_t SMEM = 1024 + (size_t)STAGES * STAGE_BYTES + 256;
 };
 
-template <int TILE_T>
+template <int TILE_T, typename MAPS>
 __global__ void __launch_bounds__(THREADS)
-gemm_wx_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x, GemmParams p) {
+gemm_wx_kernel(const __grid_constant__ MAPS maps, const __grid_constant__ GemmParams p) {
   using C = Cfg<TILE_T>;
+  constexpr bool MULTI = sizeof(MAPS) != sizeof(Maps1);
   extern __shared__ char smem_raw[];
   char* smem = reinterpret_cast<char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   char* ctrl = smem + (size_t)C::STAGES * C::STAGE_BYTES;
@@ -114,9 +141,20 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
   __shared__ float sum_scratch[33];
 
   pdl_trigger();
-  const int n_tile = blockIdx.x, t_tile = blockIdx.y, split = blockIdx.z;
+  const int grid_tile = blockIdx.x, t_tile = blockIdx.y, split = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int kb_total = (p.K + BK - 1) / BK;
+  const bool chained = MULTI && p.segments == 0;
+  const int kb_total = chained ? p.kb_all : (p.K + BK - 1) / BK;
+  int which = 0;        // beside: the product of this block's row tile
+  if (MULTI && !chained)
+    for (int s = 1; s < p.segments; ++s)
+      if (grid_tile >= p.seg[s].tile0) which = s;
+  const bool beside = MULTI && !chained;
+  const int n_tile = beside ? grid_tile - p.seg[which].tile0 : grid_tile;
+  const int N = beside ? p.seg[which].N : p.N;
+  // slice kb of K lies in pair `pair_of(kb)`, there at column `col_of(kb)`
+  auto pair_of = [&](int kb) { return !MULTI ? 0 : (chained ? (kb >= p.kb_first ? 1 : 0) : which); };
+  auto col_of = [&](int kb) { return (chained && kb >= p.kb_first ? kb - p.kb_first : kb) * BK; };
   const int per = (kb_total + p.splits - 1) / p.splits;
   const int kb0 = split * per;
   const int nkb = max(0, min(kb_total, kb0 + per) - kb0);
@@ -148,12 +186,12 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
     for (int i = 0; i < pre; ++i) {
       const uint32_t bar = smem_u32(&full[i]);
       mbar_expect_tx(bar, C::STAGE_BYTES);
-      tma_load_2d(smem_u32(smem + (size_t)i * C::STAGE_BYTES), &map_w, bar, (kb0 + i) * BK, n_tile * TILE_N);
+      tma_load_2d(smem_u32(smem + (size_t)i * C::STAGE_BYTES), &maps.w[pair_of(kb0 + i)], bar, col_of(kb0 + i), n_tile * TILE_N);
     }
     pdl_wait();
     for (int i = 0; i < pre; ++i)
-      tma_load_2d(smem_u32(smem + (size_t)i * C::STAGE_BYTES + W_STAGE_BYTES), &map_x, smem_u32(&full[i]),
-                  (kb0 + i) * BK, t_tile * TILE_T);
+      tma_load_2d(smem_u32(smem + (size_t)i * C::STAGE_BYTES + W_STAGE_BYTES), &maps.x[pair_of(kb0 + i)], smem_u32(&full[i]),
+                  col_of(kb0 + i), t_tile * TILE_T);
     int armed = pre;
     for (int i = pre; i < nkb; ++i) {
       const int s = i % C::STAGES;
@@ -162,8 +200,8 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
       const uint32_t bar = smem_u32(&full[s]);
       mbar_expect_tx(bar, C::STAGE_BYTES);
       char* stage = smem + (size_t)s * C::STAGE_BYTES;
-      tma_load_2d(smem_u32(stage), &map_w, bar, (kb0 + i) * BK, n_tile * TILE_N);
-      tma_load_2d(smem_u32(stage + W_STAGE_BYTES), &map_x, bar, (kb0 + i) * BK, t_tile * TILE_T);
+      tma_load_2d(smem_u32(stage), &maps.w[pair_of(kb0 + i)], bar, col_of(kb0 + i), n_tile * TILE_N);
+      tma_load_2d(smem_u32(stage + W_STAGE_BYTES), &maps.x[pair_of(kb0 + i)], bar, col_of(kb0 + i), t_tile * TILE_T);
       armed = i + 1;
     }
     timeline_mark(2);      // all loads issued
@@ -243,6 +281,11 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
     }
     const float wn = (epi && n < p.N) ? p.norm_w[n] : 0.f;
     const float rs = (epi && n < p.N && p.res_scale.ptr != nullptr) ? p.res_scale[n] : 1.f;
+    float wn2 = 0.f, bn = 0.f;
+    if (MULTI && epi && n < p.N) {
+      if (p.hprime2 != nullptr) wn2 = p.norm_w2[n];
+      if (p.bias.ptr != nullptr) bn = p.bias[n];
+    }
     cluster_arrive();
     cluster_wait();
     for (int j = split; j < TILE_T && t0 + j < p.M; j += p.splits) {
@@ -257,9 +300,14 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
 #pragma unroll
         for (int s = 0; s < 8; ++s)
           if (s < p.splits) sum += part[s];
+        if (MULTI) {
+          sum += bn;
+          if (p.row_factor != nullptr) sum = fmaf(p.row_factor[m], __bfloat162float(p.row_src[(size_t)m * p.N + n]), sum);
+        }
         const float v = p.residual[(size_t)m * p.N + n] + sum * rs;
         p.residual[(size_t)m * p.N + n] = v;
         p.hprime[(size_t)m * p.N + n] = __float2bfloat16_rn(v * wn);
+        if (MULTI && p.hprime2 != nullptr) p.hprime2[(size_t)m * p.N + n] = __float2bfloat16_rn(v * wn2);
         sq = v * v;
       }
       const float total = block_sum(sq, sum_scratch);
@@ -302,7 +350,10 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
       }
     }
   } else if (p.splits == 1) {
-    const float bn = (p.bias.ptr != nullptr && n < p.N) ? p.bias[n] : 0.f;
+    const VecParam bias = beside ? p.seg[which].bias : p.bias;
+    void* const out = beside ? p.seg[which].out : p.out;
+    const int ldc = beside ? p.seg[which].ldc : p.ldc, out_f32 = beside ? p.seg[which].out_f32 : p.out_f32;
+    const float bn = (bias.ptr != nullptr && n < N) ? bias[n] : 0.f;
 #pragma unroll 1
     for (int c = 0; c < TILE_T; c += 8) {
       float v[8];
@@ -317,19 +368,19 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
       }
 #pragma unroll
       for (int i = 0; i < 8; ++i) v[i] += bn;
-      if (epi && n < p.N) {
+      if (epi && n < N) {
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
           const int m = t0 + c + i;
           if (m < p.M) {
-            if (p.out_f32) static_cast<float*>(p.out)[(size_t)m * p.ldc + n] = v[i];
-            else static_cast<bf16*>(p.out)[(size_t)m * p.ldc + n] = __float2bfloat16_rn(v[i]);
+            if (out_f32) static_cast<float*>(out)[(size_t)m * ldc + n] = v[i];
+            else static_cast<bf16*>(out)[(size_t)m * ldc + n] = __float2bfloat16_rn(v[i]);
           }
         }
       }
     }
   } else {
-    const int tiles = gridDim.x * gridDim.y, tile = t_tile * gridDim.x + n_tile;
+    const int tiles = gridDim.x * gridDim.y, tile = t_tile * gridDim.x + grid_tile;
     float* mine = p.partials + ((size_t)split * tiles + tile) * (TILE_T * TILE_N);
 #pragma unroll 1
     for (int c = 0; c < TILE_T; c += 8) {
@@ -344,7 +395,8 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
         for (int i = 0; i < 8; ++i) mine[(c + i) * TILE_N + warp * 32 + lane] = scaled ? v[i] * row_scale[c + i] : v[i];
       }
     }
-    if (p.out != nullptr) {
+    void* const out = beside ? p.seg[which].out : p.out;
+    if (out != nullptr) {
       __threadfence();
       __syncthreads();
       if (threadIdx.x == 0) {
@@ -357,7 +409,9 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
         __threadfence();
         const float* base = p.partials + (size_t)tile * (TILE_T * TILE_N);
         const size_t split_stride = (size_t)tiles * (TILE_T * TILE_N);
-        const float bn = (p.bias.ptr != nullptr && n < p.N) ? p.bias[n] : 0.f;
+        const VecParam bias = beside ? p.seg[which].bias : p.bias;
+        const int ldc = beside ? p.seg[which].ldc : p.ldc, out_f32 = beside ? p.seg[which].out_f32 : p.out_f32;
+        const float bn = (bias.ptr != nullptr && n < N) ? bias[n] : 0.f;
         // eight columns at a time, so that eight chains of loads are in flight per thread
 #pragma unroll 1
         for (int c0 = 0; c0 < TILE_T && t0 + c0 < p.M; c0 += 8) {
@@ -369,13 +423,13 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
 #pragma unroll
             for (int i = 0; i < 8; ++i) sum[i] += __ldcg(src + i * TILE_N);
           }
-          if (n < p.N) {
+          if (n < N) {
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
               const int m = t0 + c0 + i;
               if (m < p.M) {
-                if (p.out_f32) static_cast<float*>(p.out)[(size_t)m * p.ldc + n] = sum[i];
-                else static_cast<bf16*>(p.out)[(size_t)m * p.ldc + n] = __float2bfloat16_rn(sum[i]);
+                if (out_f32) static_cast<float*>(out)[(size_t)m * ldc + n] = sum[i];
+                else static_cast<bf16*>(out)[(size_t)m * ldc + n] = __float2bfloat16_rn(sum[i]);
               }
             }
           }
@@ -405,24 +459,35 @@ bool make_map(CUtensorMap* map, const void* base, long long rows, long long K, l
             CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-template <int TILE_T>
-int launch(const CUtensorMap& mw, const CUtensorMap& mx, const GemmParams& p, dim3 grid, cudaStream_t stream) {
+template <int TILE_T, typename MAPS>
+int launch(const MAPS& maps, const GemmParams& p, dim3 grid, cudaStream_t stream) {
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(gemm_wx_kernel<TILE_T>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    cudaError_t e = cudaFuncSetAttribute(gemm_wx_kernel<TILE_T, MAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          (int)Cfg<TILE_T>::SMEM);
     if (e != cudaSuccess) return ts_fail("gemm_tcgen05: %s", cudaGetErrorString(e));
     configured = true;
   }
   if (p.residual != nullptr) {
     // the K cuts of a row tile are the blocks of one cluster
-    cudaError_t e = ts_launch_cluster(gemm_wx_kernel<TILE_T>, grid, dim3(THREADS), Cfg<TILE_T>::SMEM, stream,
-                                      dim3(1, 1, p.splits), mw, mx, p);
+    cudaError_t e = ts_launch_cluster(gemm_wx_kernel<TILE_T, MAPS>, grid, dim3(THREADS), Cfg<TILE_T>::SMEM, stream,
+                                      dim3(1, 1, p.splits), maps, p);
     if (e != cudaSuccess) return ts_fail("gemm_tcgen05 (clusters of %d): %s", p.splits, cudaGetErrorString(e));
     return 0;
   }
-  TS_LAUNCH("gemm_tcgen05", gemm_wx_kernel<TILE_T>, grid, THREADS, Cfg<TILE_T>::SMEM, stream, mw, mx, p);
+  TS_LAUNCH("gemm_tcgen05", (gemm_wx_kernel<TILE_T, MAPS>), grid, THREADS, Cfg<TILE_T>::SMEM, stream, maps, p);
   return 0;
+}
+
+int tile_tokens(int M) { return M <= 16 ? 16 : (M <= 32 ? 32 : (M <= 64 ? 64 : 128)); }
+
+// the kernels with several operand pairs are built for up to 64 tokens
+int launch_multi(int tile_t, const Maps3& maps, const GemmParams& p, dim3 grid, cudaStream_t stream) {
+  switch (tile_t) {
+    case 16: return launch<16>(maps, p, grid, stream);
+    case 32: return launch<32>(maps, p, grid, stream);
+    default: return launch<64>(maps, p, grid, stream);
+  }
 }
 
 }  // namespace
@@ -507,11 +572,11 @@ int gemm_tiled(const void* x, const void* w, void* out, int M, int N, int K, lon
   TS_REQUIRE(splits >= 1 && splits <= 64, "gemm_tcgen05: splits out of range");
   TS_REQUIRE(residual != nullptr || splits == 1 || (partials && (counters || out == nullptr)), "gemm_tcgen05: split-K needs scratch and counters");
   TS_REQUIRE(residual != nullptr || out != nullptr || splits > 1, "gemm_tcgen05: without an output the partial tiles must be asked for (splits > 1)");
-  const int tile_t = M <= 16 ? 16 : (M <= 32 ? 32 : (M <= 64 ? 64 : 128));
-  CUtensorMap mw, mx;
-  TS_REQUIRE(make_map(&mw, w, N, K, ldw, TILE_N), "gemm_tcgen05: cuTensorMapEncodeTiled failed for the weights");
-  TS_REQUIRE(make_map(&mx, x, M, K, ldx, tile_t), "gemm_tcgen05: cuTensorMapEncodeTiled failed for the activations");
-  GemmParams p;
+  const int tile_t = tile_tokens(M);
+  Maps1 maps;
+  TS_REQUIRE(make_map(&maps.w[0], w, N, K, ldw, TILE_N), "gemm_tcgen05: cuTensorMapEncodeTiled failed for the weights");
+  TS_REQUIRE(make_map(&maps.x[0], x, M, K, ldx, tile_t), "gemm_tcgen05: cuTensorMapEncodeTiled failed for the activations");
+  GemmParams p = {};
   p.out = out; p.partials = partials; p.counters = counters;
   p.M = M; p.N = N; p.K = K; p.ldc = (int)ldc; p.splits = splits; p.out_f32 = out_f32;
   p.x_sumsq = x_sumsq; p.x_tiles = x_tiles; p.x_eps = x_eps;
@@ -523,10 +588,81 @@ int gemm_tiled(const void* x, const void* w, void* out, int M, int N, int K, lon
   p.res_scale = VecParam{res_scale, res_scale_is_f32};
   dim3 grid((N + TILE_N - 1) / TILE_N, (M + tile_t - 1) / tile_t, splits);
   switch (tile_t) {
-    case 16: return launch<16>(mw, mx, p, grid, stream);
-    case 32: return launch<32>(mw, mx, p, grid, stream);
-    case 64: return launch<64>(mw, mx, p, grid, stream);
-    default: return launch<128>(mw, mx, p, grid, stream);
+    case 16: return launch<16>(maps, p, grid, stream);
+    case 32: return launch<32>(maps, p, grid, stream);
+    case 64: return launch<64>(maps, p, grid, stream);
+    default: return launch<128>(maps, p, grid, stream);
   }
 }
 }  // namespace
+
+// `count` (1 to 3) products side by side in one launch, for up to 64 tokens: out[i] [M, N[i]] (leading dimension
+// ldc[i], float where f32[i]) = x[i] [M, K] w[i]^T (+ bias[i]); all have the same K.  x_sumsq (up to 16 tokens): the
+// rows of every x[i] lack one and the same RMSNorm factor, as for ts_gemm_tcgen05_fused.  splits > 1 needs scratch
+// for the sum of the products' row tiles (as one product of that many rows) and counters.
+TS_EXPORT int ts_gemm_tcgen05_beside(int count, const void* const* x, const void* const* w, void* const* out, const int* N,
+                                     const long long* ldx, const long long* ldw, const long long* ldc, const int* f32,
+                                     const void* const* bias, const int* bias_is_f32, int M, int K, int splits, float* partials,
+                                     int* counters, const float* x_sumsq, int x_tiles, float x_eps, cudaStream_t stream) {
+  TS_REQUIRE(count >= 1 && count <= MAX_SEGMENTS && M > 0 && M <= 64 && K > 0 && K % 8 == 0, "gemm_tcgen05: %d products of %d tokens and K %d side by side", count, M, K);
+  TS_REQUIRE(x_sumsq == nullptr || (x_tiles > 0 && M <= SUMSQ_STRIDE), "gemm_tcgen05: the scaled-rows form takes up to %d tokens, got %d", SUMSQ_STRIDE, M);
+  TS_REQUIRE(splits >= 1 && splits <= 64 && (splits == 1 || (partials && counters)), "gemm_tcgen05: split-K needs scratch and counters");
+  const int tile_t = tile_tokens(M);
+  Maps3 maps;
+  GemmParams p = {};
+  int tiles = 0;
+  for (int i = 0; i < MAX_SEGMENTS; ++i) {
+    const int k = i < count ? i : 0;         // (the places behind the last product repeat the first)
+    TS_REQUIRE(x[k] && w[k] && out[k] && N[k] > 0 && ldx[k] % 8 == 0 && ldw[k] % 8 == 0 && ((uintptr_t)x[k] | (uintptr_t)w[k]) % 16 == 0,
+               "gemm_tcgen05: operands of product %d do not fit", k);
+    TS_REQUIRE(make_map(&maps.w[i], w[k], N[k], K, ldw[k], TILE_N) && make_map(&maps.x[i], x[k], M, K, ldx[k], tile_t),
+               "gemm_tcgen05: cuTensorMapEncodeTiled failed");
+    p.seg[i] = GemmSegment{out[k], N[k], (int)ldc[k], f32[k], tiles, VecParam{bias[k], bias_is_f32[k]}};
+    if (i < count) tiles += (N[k] + TILE_N - 1) / TILE_N;
+  }
+  p.segments = count;
+  p.partials = partials; p.counters = counters; p.M = M; p.K = K; p.splits = splits;
+  p.x_sumsq = x_sumsq; p.x_tiles = x_tiles; p.x_eps = x_eps;
+  return launch_multi(tile_t, maps, p, dim3(tiles, (M + tile_t - 1) / tile_t, splits), stream);
+}
+
+// out [M, N] = x1 [M, K1] w1^T + x2 [M, K2] w2^T (x2 null: the first alone), up to 64 tokens.  Plain: out (bfloat16 or
+// float, + bias), or with out null and splits > 1 the partial tiles only.  With residual (up to 16 tokens, splits <= 8 in
+// clusters): residual += the sum + bias + row_factor[m] * row_src[m]; hprime = bfloat16(residual * norm_w), hprime2 (or null)
+// the same with norm_w2; sumsq_out as for ts_gemm_tcgen05_fused.
+TS_EXPORT int ts_gemm_tcgen05_chain(const void* x1, const void* w1, int K1, long long ldx1, long long ldw1, const void* x2,
+                                    const void* w2, int K2, long long ldx2, long long ldw2, void* out, int M, int N,
+                                    long long ldc, int out_f32, int splits, float* partials, int* counters, const void* bias,
+                                    int bias_is_f32, float* residual, const void* norm_w, const void* norm_w2, int norm_w_is_f32,
+                                    void* hprime, void* hprime2, float* sumsq_out, const float* row_factor, const void* row_src,
+                                    cudaStream_t stream) {
+  TS_REQUIRE(M > 0 && M <= 64 && N > 0 && K1 > 0 && K1 % 8 == 0 && (x2 == nullptr || (K2 > 0 && K2 % 8 == 0 && w2)),
+             "gemm_tcgen05: a chain of K %d and %d over %d tokens", K1, K2, M);
+  TS_REQUIRE(x1 && w1 && ((uintptr_t)x1 | (uintptr_t)w1 | (uintptr_t)x2 | (uintptr_t)w2) % 16 == 0 && (ldx1 | ldw1) % 8 == 0 &&
+             (x2 == nullptr || (ldx2 | ldw2) % 8 == 0), "gemm_tcgen05: operands must be 16-byte aligned");
+  TS_REQUIRE(splits >= 1 && splits <= 64, "gemm_tcgen05: splits out of range");
+  TS_REQUIRE(residual == nullptr || (M <= SUMSQ_STRIDE && splits <= 8 && norm_w && hprime && sumsq_out && (norm_w2 == nullptr) == (hprime2 == nullptr)),
+             "gemm_tcgen05: the residual form takes up to %d tokens and 8 cuts, and needs the norm's weight and outputs", SUMSQ_STRIDE);
+  TS_REQUIRE(residual != nullptr || splits == 1 || (partials && (counters || out == nullptr)), "gemm_tcgen05: split-K needs scratch and counters");
+  TS_REQUIRE(residual != nullptr || out != nullptr || splits > 1, "gemm_tcgen05: without an output the partial tiles must be asked for (splits > 1)");
+  TS_REQUIRE(residual != nullptr || (row_factor == nullptr && (bias == nullptr || out != nullptr)), "gemm_tcgen05: row factors come with a residual, a bias with an output");
+  TS_REQUIRE(row_factor == nullptr || row_src, "gemm_tcgen05: row factors without their rows");
+  const int tile_t = tile_tokens(M);
+  Maps3 maps;
+  for (int i = 0; i < MAX_SEGMENTS; ++i) {
+    const bool second = i == 1 && x2 != nullptr;
+    TS_REQUIRE(make_map(&maps.w[i], second ? w2 : w1, N, second ? K2 : K1, second ? ldw2 : ldw1, TILE_N) &&
+               make_map(&maps.x[i], second ? x2 : x1, M, second ? K2 : K1, second ? ldx2 : ldx1, tile_t),
+               "gemm_tcgen05: cuTensorMapEncodeTiled failed");
+  }
+  GemmParams p = {};
+  p.kb_first = (K1 + BK - 1) / BK;
+  p.kb_all = p.kb_first + (x2 != nullptr ? (K2 + BK - 1) / BK : 0);
+  p.out = out; p.partials = partials; p.counters = counters;
+  p.M = M; p.N = N; p.K = p.kb_all * BK; p.ldc = (int)ldc; p.splits = splits; p.out_f32 = out_f32;
+  p.residual = residual; p.norm_w = VecParam{norm_w, norm_w_is_f32}; p.norm_w2 = VecParam{norm_w2, norm_w_is_f32};
+  p.hprime = static_cast<bf16*>(hprime); p.hprime2 = static_cast<bf16*>(hprime2); p.sumsq_out = sumsq_out;
+  p.row_factor = row_factor; p.row_src = static_cast<const bf16*>(row_src);
+  p.bias = VecParam{bias, bias_is_f32};
+  return launch_multi(tile_t, maps, p, dim3((N + TILE_N - 1) / TILE_N, (M + tile_t - 1) / tile_t, splits), stream);
+}

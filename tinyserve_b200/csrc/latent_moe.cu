@@ -197,8 +197,10 @@ __device__ __forceinline__ void route_token(const float* __restrict__ z, float* 
   }
 }
 
-// One warp, one token.  z [E] logits, corr [E] or null -> g [E]: sigmoid(z) for the chosen experts,
-// zero for the others.  scratch: 2 E + 2 groups floats of this warp's own.  Ties go to the lower number.
+// One warp, one token.  z [E] logits, corr [E] or null -> g [E]: the score for the chosen experts, zero for
+// the others; the score is sigmoid(z), or with `softmax` the softmax over all experts.  `renorm`: the chosen
+// scores are divided by their sum (+ 1e-20).  scratch: 2 E + 2 groups floats of this warp's own.  Ties go to
+// the lower number.
 __device__ __forceinline__ void warp_argmax(float& best, int& at) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) {
@@ -208,13 +210,23 @@ __device__ __forceinline__ void warp_argmax(float& best, int& at) {
   }
 }
 __device__ __forceinline__ void route_token_scored(const float* __restrict__ z, const float* __restrict__ corr, float* g,
-                                                   float* scratch, int E, int top, int groups, int keep, int lane) {
+                                                   float* scratch, int E, int top, int groups, int keep, int lane,
+                                                   int softmax = 0, int renorm = 0) {
   float* choice = scratch;            // [E] choice scores; minus infinity once taken or shut out
   float* taken = scratch + E;         // [E] 1 for a chosen expert
   float* gscore = taken + E;          // [groups]
   float* gopen = gscore + groups;     // [groups] 1 for a group whose experts may be chosen
+  float mx = 0.f, inv = 0.f;
+  if (softmax) {
+    mx = -INFINITY;
+    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
+    mx = warp_max(mx);
+    float sum = 0.f;
+    for (int e = lane; e < E; e += 32) sum += expf(z[e] - mx);
+    inv = 1.f / warp_sum(sum);
+  }
   for (int e = lane; e < E; e += 32) {
-    const float s = 1.f / (1.f + expf(-z[e]));
+    const float s = softmax ? expf(z[e] - mx) * inv : 1.f / (1.f + expf(-z[e]));
     g[e] = s;
     choice[e] = s + (corr ? corr[e] : 0.f);
     taken[e] = 0.f;
@@ -264,18 +276,57 @@ __device__ __forceinline__ void route_token_scored(const float* __restrict__ z, 
   }
   for (int e = lane; e < E; e += 32)
     if (taken[e] == 0.f) g[e] = 0.f;
+  if (renorm) {
+    __syncwarp();
+    float chosen = 0.f;
+    for (int e = lane; e < E; e += 32) chosen += g[e];
+    const float r = 1.f / (warp_sum(chosen) + 1e-20f);
+    for (int e = lane; e < E; e += 32) g[e] *= r;
+  }
 }
 
-__global__ void moe_route_scored_kernel(const float* __restrict__ logits, const float* __restrict__ corr,
-                                        float* __restrict__ gates, int num_tokens, int E, int top, int groups, int keep) {
+// The router of a step: E = experts with tensors + `identity` experts whose output is their input.
+struct Router {
+  const float* logits;     // [tokens, E]
+  const float* corr;       // [E] or null
+  int E, top, groups, keep, softmax, renorm, identity;
+  float* rest;             // [tokens]: the summed weight of the identity experts (identity > 0)
+  // the input rows of the identity experts may still lack their RMS norm factor rsqrt(sum / width + eps), sum
+  // over `sumsq` [tiles][stride] (null: they are finished): the factor then joins `rest`
+  const float* sumsq;
+  int tiles, stride, width;
+  float eps;
+};
+// One warp, one token; g [E] and scratch in shared memory.  After it (and a __syncwarp) g holds every expert's
+// weight; with `store_rest` lane 0 writes the token's entry of `rest`.
+__device__ __forceinline__ void route_scored(const Router& r, size_t t, float* g, float* scratch, int lane, bool store_rest) {
+  route_token_scored(r.logits + t * r.E, r.corr, g, scratch, r.E, r.top, r.groups, r.keep, lane, r.softmax, r.renorm);
+  if (r.identity > 0 && store_rest) {
+    __syncwarp();
+    float sum = 0.f, sq = 0.f;
+    for (int e = r.E - r.identity + lane; e < r.E; e += 32) sum += g[e];
+    sum = warp_sum(sum);
+    if (r.sumsq) {
+      for (int i = lane; i < r.tiles; i += 32) sq += __ldcg(r.sumsq + (size_t)i * r.stride + t);
+      sum *= rsqrtf(warp_sum(sq) / (float)r.width + r.eps);
+    }
+    if (lane == 0) r.rest[t] = sum;
+  }
+}
+
+// gates [tokens, E - identity]
+__global__ void moe_route_scored_kernel(Router r, float* __restrict__ gates, int num_tokens) {
   extern __shared__ float route_scratch[];
   pdl_trigger();
   pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * (blockDim.x >> 5) + warp;
   if (t >= num_tokens) return;
-  route_token_scored(logits + (size_t)t * E, corr, gates + (size_t)t * E, route_scratch + (size_t)warp * (2 * E + 2 * groups), E,
-                     top, groups, keep, lane);
+  float* g = route_scratch + (size_t)warp * (3 * r.E + 2 * r.groups);
+  route_scored(r, t, g, g + r.E, lane, true);
+  __syncwarp();
+  const int real = r.E - r.identity;
+  for (int e = lane; e < real; e += 32) gates[(size_t)t * real + e] = g[e];
 }
 
 // out[r, e * ff + j] = gated_value(a[r, e * 2 ff + j], a[r, e * 2 ff + ff + j]) * gates[r, e] (gates null: 1)
@@ -285,12 +336,16 @@ __global__ void moe_route_scored_kernel(const float* __restrict__ logits, const 
 template <typename T>
 __global__ void moe_gated_activate_kernel(const T* __restrict__ a, const float* __restrict__ gates, int E, int ff,
                                           T* __restrict__ out, int act, float limit, const float* __restrict__ logits,
-                                          const float* __restrict__ bias, int top, int renorm) {
-  extern __shared__ float routed[];      // [E] when the kernel routes
+                                          const float* __restrict__ bias, int top, int renorm, Router router) {
+  extern __shared__ float routed[];      // [E] when the kernel routes (with a scored router: its scratch behind it)
   pdl_trigger();
   pdl_wait();
   const size_t r = blockIdx.x;
-  if (logits) {
+  if (router.logits) {
+    if (threadIdx.x < 32) route_scored(router, r, routed, routed + router.E, threadIdx.x, blockIdx.y == 0);
+    __syncthreads();
+    gates = routed - r * E;
+  } else if (logits) {
     if (threadIdx.x < 32) route_token(logits + r * E, routed, E, top, threadIdx.x, renorm, bias);
     __syncthreads();
     gates = routed - r * E;              // the loop below indexes gates[r * E + e]
@@ -427,9 +482,10 @@ __global__ void moe_gather_kernel(const T* __restrict__ x, const int* __restrict
 }
 
 // out[t] = sum_e gates[t, e] * y[pair_row[t, e]] over the experts the token chose, in expert order
+// (+ rest[t] * h[t], the identity experts, with rest)
 template <typename T, bool VEC>
 __global__ void moe_combine_kernel(const T* __restrict__ y, const float* __restrict__ gates, const int* __restrict__ pair_row,
-                                   T* __restrict__ out, int E, int n) {
+                                   T* __restrict__ out, int E, int n, const float* __restrict__ rest, const T* __restrict__ h) {
   pdl_trigger();
   pdl_wait();
   const size_t t = blockIdx.x;
@@ -458,6 +514,12 @@ __global__ void moe_combine_kernel(const T* __restrict__ y, const float* __restr
 #pragma unroll
         for (int i = 0; i < N; ++i) acc[i] = fmaf(weights[k], v[i], acc[i]);
       }
+      if (rest) {
+        float v[N];
+        chunk_load<T>(h + t * n + (size_t)c * N, v);
+#pragma unroll
+        for (int i = 0; i < N; ++i) acc[i] = fmaf(rest[t], v[i], acc[i]);
+      }
       chunk_store<T>(out + t * n + (size_t)c * N, acc);
     }
   } else {
@@ -467,6 +529,7 @@ __global__ void moe_combine_kernel(const T* __restrict__ y, const float* __restr
         const int row = pair_row[t * E + e];
         if (row >= 0) acc = fmaf(gates[t * E + e], to_f32<T>(y[(size_t)row * n + c]), acc);
       }
+      if (rest) acc = fmaf(rest[t], to_f32<T>(h[t * n + c]), acc);
       out[t * n + c] = from_f32<T>(acc);
     }
   }
@@ -606,35 +669,67 @@ TS_EXPORT int ts_moe_route(const float* logits, float* gates, int num_tokens, in
   return 0;
 }
 
-TS_EXPORT int ts_moe_route_scored(const float* logits, const float* correction, float* gates, int num_tokens, int E, int top,
-                                  int groups, int keep, cudaStream_t stream) {
-  TS_REQUIRE(num_tokens > 0 && E > 0 && top > 0 && top <= E && logits && gates, "moe_route_scored: %d of %d experts", top, E);
-  TS_REQUIRE(groups >= 1 && E % groups == 0 && keep >= 1 && keep <= groups && top <= keep * (E / groups),
-             "moe_route_scored: %d experts in %d groups, %d kept, %d chosen", E, groups, keep, top);
-  const int warps = 4;
-  const size_t smem = (size_t)warps * (2 * E + 2 * groups) * sizeof(float);
-  TS_REQUIRE(smem <= 48 * 1024, "moe_route_scored: %d experts are too many", E);
-  TS_LAUNCH("moe_route_scored", moe_route_scored_kernel, (num_tokens + warps - 1) / warps, warps * 32, smem, stream, logits,
-            correction, gates, num_tokens, E, top, groups, keep);
+static int check_router(const Router& r) {
+  TS_REQUIRE(r.E > 0 && r.top > 0 && r.top <= r.E && r.identity >= 0 && r.identity < r.E && r.logits, "moe router: %d of %d experts (%d of them identity)", r.top, r.E, r.identity);
+  TS_REQUIRE(r.groups >= 1 && r.E % r.groups == 0 && r.keep >= 1 && r.keep <= r.groups && r.top <= r.keep * (r.E / r.groups),
+             "moe router: %d experts in %d groups, %d kept, %d chosen", r.E, r.groups, r.keep, r.top);
+  TS_REQUIRE(r.identity == 0 || r.rest, "moe router: identity experts need a place for their weight");
+  TS_REQUIRE(r.sumsq == nullptr || (r.tiles > 0 && r.stride > 0 && r.width > 0), "moe router: sums of squares without their sizes");
   return 0;
+}
+
+// logits [tokens, E]; the last `identity` of the E experts have no tensors: gates [tokens, E - identity], rest [tokens]
+TS_EXPORT int ts_moe_route_scored(const float* logits, const float* correction, float* gates, int num_tokens, int E, int top,
+                                  int groups, int keep, int softmax, int renorm, int identity, float* rest, cudaStream_t stream) {
+  const Router r{logits, correction, E, top, groups, keep, softmax, renorm, identity, rest, nullptr, 0, 0, 0, 0.f};
+  TS_REQUIRE(num_tokens > 0 && gates, "moe_route_scored: empty input");
+  if (int e = check_router(r)) return e;
+  const int warps = 4;
+  const size_t smem = (size_t)warps * (3 * E + 2 * groups) * sizeof(float);
+  TS_REQUIRE(smem <= 48 * 1024, "moe_route_scored: %d experts are too many", E);
+  TS_LAUNCH("moe_route_scored", moe_route_scored_kernel, (num_tokens + warps - 1) / warps, warps * 32, smem, stream, r, gates,
+            num_tokens);
+  return 0;
+}
+
+// The activation of all experts' rows with the scored router inside: a [rows, (E - identity) 2 ff]; one launch for
+// scores, choice, weights and activation.  sumsq (or null): see Router.
+static int moe_gated_activate_impl(int dtype, const void* a, const float* gates, int rows, int E, int ff, void* out, int act,
+                                   float limit, const float* logits, const float* bias, int top, int renorm, const Router& router,
+                                   size_t smem, cudaStream_t stream);
+TS_EXPORT int ts_moe_gated_activate_scored(int dtype, const void* a, int rows, int E, int ff, void* out, int act, float limit,
+                                           const float* logits, const float* correction, int top, int groups, int keep, int softmax,
+                                           int renorm, int identity, float* rest, const float* sumsq, int tiles, int stride,
+                                           int width, float eps, cudaStream_t stream) {
+  const Router r{logits, correction, E, top, groups, keep, softmax, renorm, identity, rest, sumsq, tiles, stride, width, eps};
+  if (int e = check_router(r)) return e;
+  const size_t smem = (size_t)(3 * E + 2 * groups) * sizeof(float);
+  TS_REQUIRE(smem <= 48 * 1024, "moe_gated_activate: %d experts are too many", E);
+  return moe_gated_activate_impl(dtype, a, nullptr, rows, E - identity, ff, out, act, limit, nullptr, nullptr, 0, 0, r, smem, stream);
 }
 
 TS_EXPORT int ts_moe_gated_activate(int dtype, const void* a, const float* gates, int rows, int E, int ff, void* out,
                                     int act, float limit, const float* logits, const float* bias, int top, int renorm,
                                     cudaStream_t stream) {
-  TS_REQUIRE(rows > 0 && E > 0 && ff > 0 && a && out, "moe_gated_activate: empty input");
   TS_REQUIRE(!(gates && logits) && (logits == nullptr || (top > 0 && top <= E && E <= 8192)), "moe_gated_activate: gates or logits with top of %d experts", E);
-  const size_t smem = logits ? (size_t)E * sizeof(float) : 0;
+  return moe_gated_activate_impl(dtype, a, gates, rows, E, ff, out, act, limit, logits, bias, top, renorm, Router{},
+                                 logits ? (size_t)E * sizeof(float) : 0, stream);
+}
+
+static int moe_gated_activate_impl(int dtype, const void* a, const float* gates, int rows, int E, int ff, void* out, int act,
+                                   float limit, const float* logits, const float* bias, int top, int renorm, const Router& router,
+                                   size_t smem, cudaStream_t stream) {
+  TS_REQUIRE(rows > 0 && E > 0 && ff > 0 && a && out, "moe_gated_activate: empty input");
   TS_REQUIRE(act >= 0 && act < ACT_COUNT && (act != ACT_BOUNDED_SWISH || limit > 0.f), "moe_gated_activate: activation %d", act);
   // a row's columns over several blocks (four elements a thread), so that a step of few rows still fills the SMs
   const long long tiles = ((long long)E * ff + 1023) / 1024;
   const dim3 grid(rows, (unsigned)(tiles < 64 ? tiles : 64));
   if (dtype == TS_F32)
     TS_LAUNCH("moe_gated_activate", moe_gated_activate_kernel<float>, grid, 256, smem, stream, (const float*)a, gates, E, ff, (float*)out, act, limit,
-              logits, bias, top, renorm);
+              logits, bias, top, renorm, router);
   else if (dtype == TS_BF16)
     TS_LAUNCH("moe_gated_activate", moe_gated_activate_kernel<__nv_bfloat16>, grid, 256, smem, stream, (const __nv_bfloat16*)a, gates, E, ff,
-              (__nv_bfloat16*)out, act, limit, logits, bias, top, renorm);
+              (__nv_bfloat16*)out, act, limit, logits, bias, top, renorm, router);
   else return ts_fail("moe_gated_activate: unknown dtype %d", dtype);
   return 0;
 }
@@ -684,18 +779,20 @@ TS_EXPORT int ts_moe_gather(int dtype, const void* x, const int* row_token, void
   return 0;
 }
 
+// rest [tokens] and h [tokens, n] (or both null): rest[t] * h[t] joins the sum
 TS_EXPORT int ts_moe_combine(int dtype, const void* y, const float* gates, const int* pair_row, void* out, int num_tokens, int E,
-                             int n, cudaStream_t stream) {
+                             int n, const float* rest, const void* h, cudaStream_t stream) {
+  TS_REQUIRE((rest == nullptr) == (h == nullptr), "moe_combine: the rest's weights come with its rows");
   TS_REQUIRE(num_tokens > 0 && E > 0 && n > 0 && y && gates && pair_row && out, "moe_combine: empty input");
   const int threads = n >= 2048 ? 256 : 128;
   // (a token of more than 32 experts takes the plain form)
-  const bool vec = ((uintptr_t)y | (uintptr_t)out) % 16 == 0 && n % (dtype == TS_F32 ? 4 : 8) == 0 && E <= 32;
+  const bool vec = ((uintptr_t)y | (uintptr_t)out | (uintptr_t)h) % 16 == 0 && n % (dtype == TS_F32 ? 4 : 8) == 0 && E <= 32;
   if (dtype == TS_F32) {
-    if (vec) TS_LAUNCH("moe_combine", (moe_combine_kernel<float, true>), num_tokens, threads, 0, stream, (const float*)y, gates, pair_row, (float*)out, E, n);
-    else TS_LAUNCH("moe_combine", (moe_combine_kernel<float, false>), num_tokens, threads, 0, stream, (const float*)y, gates, pair_row, (float*)out, E, n);
+    if (vec) TS_LAUNCH("moe_combine", (moe_combine_kernel<float, true>), num_tokens, threads, 0, stream, (const float*)y, gates, pair_row, (float*)out, E, n, rest, (const float*)h);
+    else TS_LAUNCH("moe_combine", (moe_combine_kernel<float, false>), num_tokens, threads, 0, stream, (const float*)y, gates, pair_row, (float*)out, E, n, rest, (const float*)h);
   } else if (dtype == TS_BF16) {
-    if (vec) TS_LAUNCH("moe_combine", (moe_combine_kernel<__nv_bfloat16, true>), num_tokens, threads, 0, stream, (const __nv_bfloat16*)y, gates, pair_row, (__nv_bfloat16*)out, E, n);
-    else TS_LAUNCH("moe_combine", (moe_combine_kernel<__nv_bfloat16, false>), num_tokens, threads, 0, stream, (const __nv_bfloat16*)y, gates, pair_row, (__nv_bfloat16*)out, E, n);
+    if (vec) TS_LAUNCH("moe_combine", (moe_combine_kernel<__nv_bfloat16, true>), num_tokens, threads, 0, stream, (const __nv_bfloat16*)y, gates, pair_row, (__nv_bfloat16*)out, E, n, rest, (const __nv_bfloat16*)h);
+    else TS_LAUNCH("moe_combine", (moe_combine_kernel<__nv_bfloat16, false>), num_tokens, threads, 0, stream, (const __nv_bfloat16*)y, gates, pair_row, (__nv_bfloat16*)out, E, n, rest, (const __nv_bfloat16*)h);
   } else {
     return ts_fail("moe_combine: unknown dtype %d", dtype);
   }

@@ -7,6 +7,8 @@
 //  * ts_causal_conv: y_t = (x_t +) (bias +) sum_j w[:, j] x_(t - taps + 1 + j) per channel, zeros
 //    before a sequence's start, optionally through silu.  The last taps - 1 inputs of every
 //    request live in its state slot and are replaced at the end of the step.
+//  * ts_conv_heads_kvwrite: the same convolution on the rows of a fused q/k/v projection, whose results
+//    go straight to padded query rows (times a factor per head) and to the token's cache slot.
 //  * ts_group_norm / ts_group_norm_add: RMS norm of every one of `groups` equal consecutive parts
 //    of a row, times a weight; written out (optionally only some rows), or added to the 32-bit
 //    residual.
@@ -138,6 +140,162 @@ __global__ void __launch_bounds__(CONV_THREADS) causal_conv_kernel(ConvParams p)
       st[(size_t)i * p.C] = v;
     }
   }
+}
+
+// ------------------------------------------------------------------ causal convolution of q, k, v + cache write
+// The rows x [T, H dim (q) | G dim (k) | G vdim (v)] of a fused projection pass the convolution and leave as what
+// the attention kernels read: query rows [T, H, stored] (times one factor per head), keys and values at the cache
+// slots of their tokens, heads padded with zeros to `stored`.  G = 0: queries only (the keys and values are
+// another layer's).  A thread owns VEC neighbouring columns of a stored head over CONV_TILE tokens of one request;
+// the block of a request's first tile also replaces the request's state, as in causal_conv_kernel.
+struct ConvHeads {
+  const void* x; long long ldx;
+  VecParam w;                       // [channels, TAPS]; null (TAPS 1): the rows as they are
+  VecParam factor;                  // [H] or null
+  float* state;                     // [slots, TAPS - 1, channels]
+  const int* state_slots; const int* fresh; const int* cu_q;
+  int H, G, dim, vdim, stored, page_size, channels;
+  void* q_out; void* k_cache; void* v_cache;
+  const int* slot_mapping;
+};
+constexpr int CONV_BATCH = 8;        // tokens whose loads are in flight together
+
+template <typename T, int VEC> struct Pack;
+template <> struct Pack<float, 1> {
+  static __device__ __forceinline__ void load(const float* p, float (&v)[1]) { v[0] = *p; }
+  static __device__ __forceinline__ void store(float* p, const float (&v)[1]) { *p = v[0]; }
+};
+template <> struct Pack<float, 2> {
+  static __device__ __forceinline__ void load(const float* p, float (&v)[2]) {
+    const float2 q = *reinterpret_cast<const float2*>(p);
+    v[0] = q.x; v[1] = q.y;
+  }
+  static __device__ __forceinline__ void store(float* p, const float (&v)[2]) { *reinterpret_cast<float2*>(p) = make_float2(v[0], v[1]); }
+};
+template <> struct Pack<__nv_bfloat16, 1> {
+  static __device__ __forceinline__ void load(const __nv_bfloat16* p, float (&v)[1]) { v[0] = __bfloat162float(*p); }
+  static __device__ __forceinline__ void store(__nv_bfloat16* p, const float (&v)[1]) { *p = __float2bfloat16_rn(v[0]); }
+};
+template <> struct Pack<__nv_bfloat16, 2> {
+  static __device__ __forceinline__ void load(const __nv_bfloat16* p, float (&v)[2]) {
+    const __nv_bfloat162 q = *reinterpret_cast<const __nv_bfloat162*>(p);
+    v[0] = __low2float(q); v[1] = __high2float(q);
+  }
+  static __device__ __forceinline__ void store(__nv_bfloat16* p, const float (&v)[2]) {
+    *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(v[0], v[1]);
+  }
+};
+
+template <typename T, int VEC, int TAPS>
+__global__ void __launch_bounds__(CONV_THREADS) conv_heads_kvwrite_kernel(ConvHeads p) {
+  pdl_trigger();
+  constexpr int H1 = TAPS - 1;
+  const int col = (blockIdx.x * CONV_THREADS + threadIdx.x) * VEC;      // over the stored heads: q, then k, then v
+  const int head = col / p.stored, d = col % p.stored;
+  const bool is_q = head < p.H, is_v = head >= p.H + p.G;
+  const int g = is_q ? head : (is_v ? head - p.H - p.G : head - p.H);
+  const bool live = head < p.H + 2 * p.G;
+  const bool real = live && d < (is_v ? p.vdim : p.dim);                // else: a column of zeros
+  // the projection's column, which is also the convolution's channel
+  const int c = is_q ? g * p.dim + d : (is_v ? (p.H + p.G) * p.dim + g * p.vdim + d : p.H * p.dim + g * p.dim + d);
+  float w[TAPS][VEC];
+  float factor = 1.f;
+  if (real) {      // (weights are constants: fetched while the predecessor still runs)
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) w[j][e] = p.w.ptr ? p.w[(c + e) * TAPS + j] : 1.f;
+    if (is_q && p.factor.ptr) factor = p.factor[head];
+  }
+  pdl_wait();
+  const int b = blockIdx.z;
+  const int t0 = p.cu_q[b], n = p.cu_q[b + 1] - t0;
+  const int first = blockIdx.y * CONV_TILE;
+  if (first >= n || !live) return;
+  const T* x = static_cast<const T*>(p.x) + c;
+  float* st = nullptr;
+  float hist[H1 > 0 ? H1 : 1][VEC];
+  bool is_fresh = false;
+  if (H1 > 0 && real) {
+    st = p.state + (size_t)p.state_slots[b] * H1 * p.channels + c;
+    is_fresh = p.fresh[b] != 0;
+#pragma unroll
+    for (int i = 0; i < H1; ++i) {       // hist[i] = input at token first - H1 + i of this portion (before it: the state)
+      if (first == 0) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) hist[i][e] = is_fresh ? 0.f : st[(size_t)i * p.channels + e];
+      } else {
+        Pack<T, VEC>::load(x + (size_t)(t0 + first - H1 + i) * p.ldx, hist[i]);
+      }
+    }
+  }
+  const int last = min(n, first + CONV_TILE);
+  for (int tok0 = first; tok0 < last; tok0 += CONV_BATCH) {
+    float in[CONV_BATCH][VEC];
+    int slot[CONV_BATCH];
+#pragma unroll
+    for (int k = 0; k < CONV_BATCH; ++k) {
+      if (tok0 + k < last) {
+        if (real) Pack<T, VEC>::load(x + (size_t)(t0 + tok0 + k) * p.ldx, in[k]);
+        slot[k] = is_q ? 0 : p.slot_mapping[t0 + tok0 + k];
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < CONV_BATCH; ++k) {
+      if (tok0 + k >= last) break;
+      float y[VEC];
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) {
+        float acc = 0.f;
+        if (real) {
+          acc = w[H1][e] * in[k][e];
+#pragma unroll
+          for (int i = 0; i < H1; ++i) acc = fmaf(w[i][e], hist[i][e], acc);
+          acc *= factor;
+#pragma unroll
+          for (int i = 0; i + 1 < H1; ++i) hist[i][e] = hist[i + 1][e];
+          if (H1 > 0) hist[H1 - 1][e] = in[k][e];
+        }
+        y[e] = acc;
+      }
+      if (is_q) {
+        Pack<T, VEC>::store(static_cast<T*>(p.q_out) + ((size_t)(t0 + tok0 + k) * p.H + head) * p.stored + d, y);
+      } else if (slot[k] >= 0) {
+        const size_t page = slot[k] / p.page_size, in_page = slot[k] % p.page_size;
+        T* cache = static_cast<T*>(is_v ? p.v_cache : p.k_cache);
+        Pack<T, VEC>::store(cache + ((page * p.G + g) * p.page_size + in_page) * p.stored + d, y);
+      }
+    }
+  }
+  if (H1 > 0 && first == 0 && real) {
+    // new state: inputs at tokens n - H1 .. n - 1; tokens below 0 are the old state's row i + n, which an ascending
+    // walk has not overwritten yet
+#pragma unroll
+    for (int i = 0; i < H1; ++i) {
+      const int tok = n - H1 + i;
+      float v[VEC];
+      if (tok >= 0) {
+        Pack<T, VEC>::load(x + (size_t)(t0 + tok) * p.ldx, v);
+      } else {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) v[e] = is_fresh ? 0.f : st[(size_t)(i + n) * p.channels + e];
+      }
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) st[(size_t)i * p.channels + e] = v[e];
+    }
+  }
+}
+
+template <typename T, int VEC>
+int launch_conv_heads(const ConvHeads& p, int taps, dim3 grid, cudaStream_t stream) {
+  switch (taps) {
+#define TS_CONV_CASE(N) \
+    case N: TS_LAUNCH("conv_heads_kvwrite", (conv_heads_kvwrite_kernel<T, VEC, N>), grid, CONV_THREADS, 0, stream, p); break;
+    TS_CONV_CASE(1) TS_CONV_CASE(2) TS_CONV_CASE(3) TS_CONV_CASE(4) TS_CONV_CASE(5) TS_CONV_CASE(6) TS_CONV_CASE(7)
+    TS_CONV_CASE(8)
+#undef TS_CONV_CASE
+  }
+  return 0;
 }
 
 // ------------------------------------------------------------------ RMS norm in groups
@@ -453,6 +611,27 @@ TS_EXPORT int ts_causal_conv(const void* x, long long ldx, int x_is_f32, void* y
 #undef TS_CONV_CASE
   }
   return 0;
+}
+
+// x [T, H dim | G dim | G vdim]; w [channels, taps] or null (taps 1); factor [H] or null; G 0: queries only
+TS_EXPORT int ts_conv_heads_kvwrite(int is_f32, const void* x, long long ldx, const void* w, int w_is_f32, int taps,
+                                    const void* factor, int factor_is_f32, float* state, const int* state_slots,
+                                    const int* fresh, const int* cu_q, int num_requests, int max_q_len, int H, int G, int dim,
+                                    int vdim, int stored, void* q_out, void* k_cache, void* v_cache, const int* slot_mapping,
+                                    int page_size, cudaStream_t stream) {
+  TS_REQUIRE(num_requests > 0 && max_q_len > 0 && H > 0 && G >= 0 && dim > 0 && vdim > 0 && stored >= dim && stored >= vdim,
+             "conv_heads_kvwrite: sizes do not fit");
+  TS_REQUIRE(taps >= 1 && taps <= CONV_MAX_TAPS && (w || taps == 1), "conv_heads_kvwrite: 1 to %d taps, got %d", CONV_MAX_TAPS, taps);
+  TS_REQUIRE(x && q_out && (taps == 1 || state) && state_slots && fresh && cu_q, "conv_heads_kvwrite: a null operand");
+  TS_REQUIRE(G == 0 || (k_cache && v_cache && slot_mapping && page_size > 0), "conv_heads_kvwrite: no cache to write");
+  ConvHeads p{x, ldx, VecParam{w, w_is_f32}, VecParam{factor, factor_is_f32}, state, state_slots, fresh, cu_q, H, G, dim, vdim, stored,
+              page_size, H * dim + G * (dim + vdim), q_out, k_cache, v_cache, slot_mapping};
+  const bool even = dim % 2 == 0 && vdim % 2 == 0 && stored % 2 == 0 && ldx % 2 == 0 && (uintptr_t)x % 8 == 0;
+  const int cols = (H + 2 * G) * stored / (even ? 2 : 1);
+  const dim3 grid((cols + CONV_THREADS - 1) / CONV_THREADS, (max_q_len + CONV_TILE - 1) / CONV_TILE, num_requests);
+  TS_REQUIRE(grid.y <= 65535 && grid.z <= 65535, "conv_heads_kvwrite: the step is too large");
+  if (is_f32) return even ? launch_conv_heads<float, 2>(p, taps, grid, stream) : launch_conv_heads<float, 1>(p, taps, grid, stream);
+  return even ? launch_conv_heads<__nv_bfloat16, 2>(p, taps, grid, stream) : launch_conv_heads<__nv_bfloat16, 1>(p, taps, grid, stream);
 }
 
 // rows null: every row of x [num_out, n]; else out[o] = norm(x[rows[o]])

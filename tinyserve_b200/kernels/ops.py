@@ -163,10 +163,11 @@ class PendingProduct:
     (the K cuts of a row tile are a thread-block cluster; they add their partial sums through
     distributed shared memory, add the residual and leave a ScaledRows).  For many tokens
     (``wide``) the paired kernel has the same form.  Any other consumer calls ``partials()`` or
-    ``materialize()`` and gets the ordinary product."""
+    ``materialize()`` and gets the ordinary product.  ``bias`` [N] (or None) belongs to the product;
+    partial tiles have no place for it."""
 
-    def __init__(self, x, weight, wide=False):
-        self.x, self.weight, self.wide = x, weight, wide         # wide: many tokens, the paired kernel
+    def __init__(self, x, weight, wide=False, bias=None):
+        self.x, self.weight, self.wide, self.bias = x, weight, wide, bias         # wide: many tokens, the paired kernel
         self.shape = (x.shape[0], weight.shape[0])
         self.dtype, self.device = x.dtype, x.device
 
@@ -175,14 +176,19 @@ class PendingProduct:
         return min(gemm_splits(M, self.weight.shape[0], K, partials=True), FUSED_MAX_SPLITS)
 
     def partials(self):
-        if not self.wide and self.splits() > 1:
+        if not self.wide and self.bias is None and self.splits() > 1:
             return _linear_tcgen05(self.x, self.weight, False, partials_only=True)
         return self.materialize()
 
     def materialize(self):
         if self.wide:
             return _linear_pair(self.x, self.weight)
-        return _linear_tcgen05(self.x, self.weight, False)
+        return _linear_tcgen05(self.x, self.weight, False, bias=self.bias)
+
+    @property
+    def fits_residual_form(self):
+        """The product may add the residual itself: few tokens (or the paired kernel), no bias."""
+        return self.bias is None and (self.wide or self.x.shape[0] <= FUSED_MAX_TOKENS)
 
 
 class ScaledRows:
@@ -219,7 +225,7 @@ _NO_SCALE = (c_void_p(0), c_int(0), c_float(0.0))
 
 def materialize(x):
     """An ordinary tensor from what a product, a norm or a block returned."""
-    return x.materialize() if isinstance(x, (SplitPartials, PendingProduct, ScaledRows, PairSum, NormedAddend, ColumnScaled)) else x
+    return x.materialize() if isinstance(x, (SplitPartials, PendingProduct, ScaledRows, PairSum, NormedAddend, ColumnScaled, BranchSum, RowsAdded)) else x
 
 
 def launch_count() -> int:
@@ -617,17 +623,19 @@ def add_rmsnorm(x, residual, weight, eps, out_dtype, rows=None, scaled_ok=False)
     ``rows`` (int32) only those rows are normalised and returned, and the residual is left as it
     is.  With ``scaled_ok`` the caller takes a ScaledRows as well (it hands it to ``linear``)."""
     x_scale = None
+    if isinstance(x, (BranchSum, RowsAdded)):
+        return branch_norm(x, residual, weight, None, eps, out_dtype, rows=rows, scaled_ok=scaled_ok)[0]
     if isinstance(x, ColumnScaled):
         x, x_scale = x.x, x.scale
         if isinstance(x, PendingProduct):
-            if (scaled_ok and rows is None and out_dtype == torch.bfloat16 and not x.wide and x.shape == tuple(residual.shape)
+            if (scaled_ok and rows is None and out_dtype == torch.bfloat16 and not x.wide and x.fits_residual_form and x.shape == tuple(residual.shape)
                     and residual.dtype == torch.float32 and residual.is_contiguous()
                     and x_scale.shape == (residual.shape[1],) and x_scale.is_contiguous()):
                 _cuda(residual, weight, x_scale)
                 return _product_add_residual(x, residual, weight, eps, x_scale)
             x = x.partials()
     if isinstance(x, PendingProduct):
-        if (scaled_ok and rows is None and out_dtype == torch.bfloat16 and x.shape == tuple(residual.shape)
+        if (scaled_ok and rows is None and out_dtype == torch.bfloat16 and x.fits_residual_form and x.shape == tuple(residual.shape)
                 and residual.dtype == torch.float32 and residual.is_contiguous()):
             _cuda(residual, weight)
             return _product_add_residual(x, residual, weight, eps)
@@ -852,8 +860,15 @@ def decode_splits(num_requests, max_kv_len, num_heads, num_kv_heads):
     return max(1, min(2 * num_sms() // blocks, max_kv_len // 128, 32))
 
 
+def _turn_args(turn, ctx):
+    """(cos, sin, pairs, positions) of a turn-back of the outputs (see ``paged_attention``), or nulls."""
+    if turn is None:
+        return c_void_p(0), c_void_p(0), c_int(0), c_void_p(0)
+    return _ptr(turn.cos), _ptr(turn.sin), c_int(turn.rotary_dim // 2), _ptr(ctx.positions)
+
+
 def _decode_listed(q, out, k_cache, v_cache, view, ctx, scale, window, work, keep_first=0, sinks=None, chunk=0,
-                   slopes=None, softcap=0.0):
+                   slopes=None, softcap=0.0, turn=None):
     """The one-token requests of a mixed batch, by the tensor-core decode kernel."""
     T, H, D = q.shape
     Hkv = k_cache.shape[1]
@@ -871,7 +886,7 @@ def _decode_listed(q, out, k_cache, v_cache, view, ctx, scale, window, work, kee
         c_int(view.page_size), c_int(view.block_table.stride(0)), c_float(scale), c_int(window),
         c_int(num_splits), _ptr(part_o), _ptr(part_ml), c_int(2 if cluster else 1), _ptr(work.dec_req),
         _ptr(work.dec_tok), c_int(n), c_int(0), c_int(_tma_pages(k_cache, v_cache)), c_int(keep_first), _ptr(sinks),
-        c_int(chunk), _ptr(slopes), c_float(softcap), c_int(Hkv // v_cache.shape[1]), _stream()),
+        c_int(chunk), _ptr(slopes), c_float(softcap), c_int(Hkv // v_cache.shape[1]), *_turn_args(turn, ctx), _stream()),
         2 if num_splits > 1 and not cluster else 1)
 
 
@@ -907,7 +922,7 @@ def biased_attention_backends(dtype, head_dim, page_size) -> list:
 
 
 def paged_attention(q, k_cache, v_cache, view, ctx, scale, window=0, num_splits=None, backend=None, keep_first=0,
-                    sinks=None, chunk=0, slopes=None, softcap=0.0):
+                    sinks=None, chunk=0, slopes=None, softcap=0.0, turn=None):
     """Attention of this step's queries over their requests' cached keys and values.
     ``chunk`` > 0: a query at position i sees key j <= i only if i // chunk == j // chunk (chunks
     count from position 0 of the sequence; no window beside it).  ``slopes`` float32 [H]: head h's
@@ -916,6 +931,8 @@ def paged_attention(q, k_cache, v_cache, view, ctx, scale, window=0, num_splits=
     ``sinks`` float32 [H]: head h's softmax sum holds one more term exp(sinks[h]) without key or value.
     ``softcap`` c > 0: the scaled score s becomes c tanh(s / c) (before the slopes' bias).
     A value cache of fewer heads than the key cache (Hkv / s): key head i reads value head i / s.
+    ``turn``: a rotary encoding in neighbouring pairs; every output row is turned back by its query's
+    position over the first ``turn.rotary_dim`` columns (the values in the cache were turned by theirs).
     q [T, H, D]; caches [pages, Hkv, page_size, D]; ``view`` a GroupView; ``ctx`` gives cu_q,
     kv_lens and the batch's maxima.  bfloat16 runs on the tensor cores (a decode kernel when
     every request brings one token, else a prefill kernel); float32 on the 32-bit kernel.
@@ -935,6 +952,8 @@ def paged_attention(q, k_cache, v_cache, view, ctx, scale, window=0, num_splits=
     softcap = float(softcap or 0.0)
     if softcap < 0:
         raise ValueError("paged_attention: a soft cap is positive (0: none)")
+    if turn is not None and (not turn.interleaved or turn.rotary_dim > D):
+        raise ValueError("paged_attention: outputs turn back in neighbouring pairs of the head")
     if chunk < 0 or (chunk and window > 0):
         raise ValueError("paged_attention: a chunk is positive and comes without a window")
     if slopes is not None and (slopes.dtype != torch.float32 or slopes.shape != (H,) or not slopes.is_cuda):
@@ -953,7 +972,7 @@ def paged_attention(q, k_cache, v_cache, view, ctx, scale, window=0, num_splits=
         tile_queries = prefill_tile_queries(q.dtype, H, Hkv, D, page)
         work = attention_work(ctx, tile_queries, q.device)
         if work.num_decode:
-            _decode_listed(q, out, k_cache, v_cache, view, ctx, scale, window, work, keep_first, sinks, chunk, slopes, softcap)
+            _decode_listed(q, out, k_cache, v_cache, view, ctx, scale, window, work, keep_first, sinks, chunk, slopes, softcap, turn)
         if work.num_tiles:
             _check(lib, lib.ts_paged_attention_tcgen05(
                 _ptr(q), _ptr(out), _ptr(k_cache), _ptr(v_cache), _ptr(view.block_table), _ptr(ctx.cu_q),
@@ -961,7 +980,7 @@ def paged_attention(q, k_cache, v_cache, view, ctx, scale, window=0, num_splits=
                 c_int(k_cache.shape[0]), c_int(page), c_int(view.block_table.stride(0)), c_float(scale),
                 c_int(window), _ptr(work.tile_req), _ptr(work.tile_q0), c_int(work.num_tiles),
                 c_int(tile_queries), c_int(keep_first), _ptr(sinks), c_int(chunk), _ptr(slopes), c_float(softcap),
-                c_int(v_share), _stream()))
+                c_int(v_share), *_turn_args(turn, ctx), _stream()))
         return out
     if num_splits is None:
         if decode:
@@ -989,7 +1008,7 @@ def paged_attention(q, k_cache, v_cache, view, ctx, scale, window=0, num_splits=
             tile_queries = rows // group if group < rows else 1
             work = attention_work(ctx, tile_queries, q.device)
             if work.num_decode:
-                _decode_listed(q, out, k_cache, v_cache, view, ctx, scale, window, work, keep_first, sinks, chunk, slopes, softcap)
+                _decode_listed(q, out, k_cache, v_cache, view, ctx, scale, window, work, keep_first, sinks, chunk, slopes, softcap, turn)
             if not work.num_tiles:
                 return out
             tile_req, tile_q0, num_tiles = work.tile_req, work.tile_q0, work.num_tiles
@@ -1000,7 +1019,7 @@ def paged_attention(q, k_cache, v_cache, view, ctx, scale, window=0, num_splits=
             c_int(window), c_int(num_splits), _ptr(part_o), _ptr(part_ml),
             c_int((2 if cluster else 1) if decode else 0), _ptr(tile_req), _ptr(tile_q0), c_int(num_tiles), c_int(tile_queries),
             c_int(_tma_pages(k_cache, v_cache)), c_int(keep_first), _ptr(sinks), c_int(chunk), _ptr(slopes),
-            c_float(softcap), c_int(v_share), _stream()),
+            c_float(softcap), c_int(v_share), *_turn_args(turn, ctx), _stream()),
             launches)
         return out
     lib = _attention(D)
@@ -1009,7 +1028,7 @@ def paged_attention(q, k_cache, v_cache, view, ctx, scale, window=0, num_splits=
         _ptr(ctx.cu_q), _ptr(ctx.kv_lens), c_int(T), c_int(ctx.num_requests), c_int(ctx.max_q_len),
         c_int(H), c_int(Hkv), c_int(view.page_size), c_int(view.block_table.stride(0)),
         c_float(scale), c_int(window), c_int(num_splits), _ptr(part_o), _ptr(part_ml), c_int(keep_first),
-        _ptr(sinks), c_int(chunk), _ptr(slopes), c_float(softcap), c_int(v_share), _stream()),
+        _ptr(sinks), c_int(chunk), _ptr(slopes), c_float(softcap), c_int(v_share), *_turn_args(turn, ctx), _stream()),
         launches)
     return out
 
@@ -1087,12 +1106,12 @@ def linear(x, weight, bias=None, out_float32=False, allow_partials=False, allow_
             return PendingProduct(x, weight, wide=True)
         return _linear_pair(x, weight, out_float32, bias=bias, scale=scale)
     if x.dtype == torch.bfloat16 and _tcgen05_ok(x, weight) and (scale is None or M <= FUSED_MAX_TOKENS):
+        if allow_pending and scale is None and not out_float32:
+            return PendingProduct(x, weight, bias=bias)
         if bias is not None:
             if scale is not None:
                 x, scale = scale.materialize(), None
             return _linear_tcgen05(x, weight, out_float32, bias=bias)
-        if allow_pending and scale is None and not out_float32 and M <= FUSED_MAX_TOKENS:
-            return PendingProduct(x, weight)
         if (allow_partials or allow_pending) and not out_float32 \
                 and gemm_splits(x.shape[0], weight.shape[0], x.shape[1], partials=True) > 1:
             return _linear_tcgen05(x, weight, False, partials_only=True, scale=scale)
@@ -1190,7 +1209,7 @@ class ColumnScaled:
     to any other consumer."""
 
     def __init__(self, x, scale):
-        if isinstance(x, (PairSum, NormedAddend, ScaledRows, ColumnScaled)):
+        if isinstance(x, (PairSum, NormedAddend, ScaledRows, ColumnScaled, BranchSum, RowsAdded)):
             x = materialize(x)
         self.x, self.scale = x, scale
         self.shape, self.dtype, self.device = tuple(x.shape), x.dtype, x.device
@@ -1266,13 +1285,13 @@ def add_layernorm(x, residual, weight, eps, out_dtype, bias=None, rows=None):
     return out
 
 
-def softcap_(logits, cap):
-    """logits (float32, in place) <- cap * tanh(logits / cap)."""
+def softcap_(logits, cap, scale=1.0):
+    """logits (float32, in place) <- cap * tanh(scale * logits / cap); ``cap`` 0: scale * logits."""
     _cuda(logits)
     if logits.dtype != torch.float32 or not logits.is_contiguous():
         raise TypeError("softcap: logits are contiguous float32")
     lib = _elementwise()
-    _check(lib, lib.ts_softcap(_ptr(logits), c_longlong(logits.numel()), c_float(cap), _stream()))
+    _check(lib, lib.ts_softcap(_ptr(logits), c_longlong(logits.numel()), c_float(cap), c_float(scale), _stream()))
     return logits
 
 
@@ -1328,7 +1347,7 @@ def _columns(t):
 
 def rope_unit_kvwrite(q, k, v, positions, num_heads, num_kv_heads, dim, vdim, stored_dim, rotary=None,
                       unit_norm=False, eps=0.0, k_cache=None, v_cache=None, slot_mapping=None, page_size=0,
-                      q_weight=None, k_weight=None, pre_eps=0.0, maps=1):
+                      q_weight=None, k_weight=None, pre_eps=0.0, maps=1, value_rotary=None):
     """Rotary encoding of q and k (first ``rotary.rotary_dim`` elements of every head), then, with
     ``unit_norm``, division of every head of q and k by its root mean square over ``dim``; q goes
     to a [T, H, stored_dim] tensor (returned), k and v to the cache slots of ``slot_mapping``
@@ -1341,13 +1360,21 @@ def rope_unit_kvwrite(q, k, v, positions, num_heads, num_kv_heads, dim, vdim, st
     in q and k, v holds ``num_kv_heads`` / M heads and so does the value cache, and the returned
     query rows are arranged so that the attention kernels pair map m of a head with map m of its
     key/value head (``paged_attention`` gives key head i the value head i / M; ``map_difference``
-    reads the output in that order)."""
+    reads the output in that order).  ``value_rotary`` (neighbouring pairs, over all of ``vdim``): every
+    value is turned to its token's position before it is stored (``paged_attention(turn=)``).
+    Without ``slot_mapping`` k and v may be None."""
+    if k is None and v is None and slot_mapping is None:
+        k, v = q[:, :0], q[:, :0]
+    elif k.shape[1] != num_kv_heads * dim or v.shape[1] != num_kv_heads // maps * vdim:
+        raise ValueError("rope_unit_kvwrite: k, v do not have heads x size columns")
+    if value_rotary is not None and (not value_rotary.interleaved or value_rotary.rotary_dim != vdim):
+        raise ValueError("rope_unit_kvwrite: values turn in neighbouring pairs over their whole size")
     _cuda(q, k, v, positions, k_cache, v_cache, slot_mapping, q_weight, k_weight)
     T = q.shape[0]
     if maps < 1 or num_heads % maps or num_kv_heads % maps:
         raise ValueError("rope_unit_kvwrite: the maps do not divide the heads")
-    if q.shape[1] != num_heads * dim or k.shape[1] != num_kv_heads * dim or v.shape[1] != num_kv_heads // maps * vdim:
-        raise ValueError("rope_unit_kvwrite: q, k, v do not have heads x size columns")
+    if q.shape[1] != num_heads * dim:
+        raise ValueError("rope_unit_kvwrite: q does not have heads x size columns")
     if (q_weight is None) != (k_weight is None) or (q_weight is not None and (
             q_weight.dtype != k_weight.dtype or q_weight.shape != (dim,) or k_weight.shape != (dim,))):
         raise TypeError("rope_unit_kvwrite: q and k norm weights come together, [dim] each and alike in dtype")
@@ -1365,7 +1392,8 @@ def rope_unit_kvwrite(q, k, v, positions, num_heads, num_kv_heads, dim, vdim, st
         c_int(1 if unit_norm else 0), c_float(eps), c_int(T), c_int(num_heads), c_int(num_kv_heads), c_int(dim),
         c_int(vdim), c_int(stored_dim), _ptr(k_cache), _ptr(v_cache), _ptr(slot_mapping), c_int(page_size),
         _ptr(q_weight), _ptr(k_weight), c_int(_vec_flag(q_weight, q.dtype) if q_weight is not None else 0),
-        c_float(pre_eps), c_int(maps), _stream()))
+        c_float(pre_eps), c_int(maps), _ptr(value_rotary.cos if value_rotary is not None else None),
+        _ptr(value_rotary.sin if value_rotary is not None else None), _stream()))
     return out
 
 
@@ -1692,10 +1720,11 @@ def moe_activate_(a, gates, num_experts, logits=None, top=0):
 MOE_GROUPED_MIN_TOKENS = 256
 
 
-def moe_grouped(h, gates, up, down_side_by_side, top, gated=False, activation="silu", limit=0.0):
+def moe_grouped(h, gates, up, down_side_by_side, top, gated=False, activation="silu", limit=0.0, rest=None):
     """Mixture of experts over rows sorted by expert.  h [T, n] bfloat16; gates float32 [T, E] (zero:
     not chosen); up [E ff, n] (expert by expert); down_side_by_side [n, E ff].  Returns [T, n]:
-    sum over a token's experts of gate * W_down,e relu(W_up,e h)^2, the sum in 32-bit.  The two
+    sum over a token's experts of gate * W_down,e relu(W_up,e h)^2, the sum in 32-bit; with ``rest``
+    (float32 [T]) + rest * h (experts whose output is their input).  The two
     products over ragged row groups are the library's grouped product."""
     _cuda(h, gates, up, down_side_by_side)
     T, n = h.shape
@@ -1719,7 +1748,7 @@ def moe_grouped(h, gates, up, down_side_by_side, top, gated=False, activation="s
     y = torch.nn.functional.grouped_mm(a, down_side_by_side.view(n, E, ff).permute(1, 2, 0), offs=ends)
     out = torch.empty(T, n, dtype=h.dtype, device=h.device)
     _check(lib, lib.ts_moe_combine(c_int(_dt(y)), _ptr(y), _ptr(gates), _ptr(pair_row), _ptr(out), c_int(T), c_int(E), c_int(n),
-                                   _stream()))
+                                   _ptr(rest), _ptr(h if rest is not None else None), _stream()))
     count_launches(2)
     return out
 
@@ -1914,21 +1943,56 @@ def ssm_finish(raw, x, skip, z, weight, groups, eps, num_heads, value_dim, out_d
 
 
 # ----------------------------------------------------------------------------- experts chosen by scores with a correction
-def moe_route_scored(logits, correction, top, groups=1, keep=1):
+def _check_scored(logits, correction):
+    if logits.dtype != torch.float32 or not logits.is_contiguous():
+        raise TypeError("moe router: router logits are contiguous float32")
+    if correction is not None and (correction.dtype != torch.float32 or correction.shape != (logits.shape[1],)):
+        raise TypeError("moe router: the correction is float32 [experts]")
+
+
+def moe_route_scored(logits, correction, top, groups=1, keep=1, softmax=False, renormalize=False, identity=0):
     """float32 [T, E] router logits -> float32 [T, E] weights: s = sigmoid(z) for the ``top`` experts
     with the largest s + correction among the experts of the ``keep`` best of ``groups`` equal groups
-    of neighbours (a group's score: the sum of its two largest s + correction), zero elsewhere."""
+    of neighbours (a group's score: the sum of its two largest s + correction), zero elsewhere.
+    ``softmax``: s is the softmax over all E instead.  ``renormalize``: the chosen s are divided by their
+    sum (+ 1e-20).  ``identity`` k > 0: the last k experts have no tensors (their output is their
+    input); returns ([T, E - k] weights, [T] the summed weight of the last k)."""
     _cuda(logits, correction)
-    if logits.dtype != torch.float32 or not logits.is_contiguous():
-        raise TypeError("moe_route_scored: router logits are contiguous float32")
+    _check_scored(logits, correction)
     T, E = logits.shape
-    if correction is not None and (correction.dtype != torch.float32 or correction.shape != (E,)):
-        raise TypeError("moe_route_scored: the correction is float32 [experts]")
-    gates = torch.empty_like(logits)
+    gates = torch.empty(T, E - identity, dtype=torch.float32, device=logits.device)
+    rest = torch.empty(T, dtype=torch.float32, device=logits.device) if identity else None
     lib = _latent_moe()
     _check(lib, lib.ts_moe_route_scored(_ptr(logits), _ptr(correction), _ptr(gates), c_int(T), c_int(E), c_int(top),
-                                        c_int(groups), c_int(keep), _stream()))
-    return gates
+                                        c_int(groups), c_int(keep), c_int(1 if softmax else 0), c_int(1 if renormalize else 0),
+                                        c_int(identity), _ptr(rest), _stream()))
+    return (gates, rest) if identity else gates
+
+
+def moe_gated_activate_scored(a, logits, correction, top, groups=1, keep=1, softmax=False, renormalize=False, identity=0,
+                              activation="silu", limit=0.0, scaled=None):
+    """``moe_gated_activate`` with the router of ``moe_route_scored`` inside: a [rows, (E - identity) 2 ff],
+    logits float32 [rows, E].  Returns (activated rows, rest): ``rest`` float32 [rows] is the weight of the
+    identity experts (None without any).  ``scaled``: the ScaledRows the identity experts read; their
+    rows' missing norm factor is then part of ``rest``, which belongs to ``scaled.data``."""
+    _cuda(a, logits, correction)
+    _check_scored(logits, correction)
+    code, limit = activation_code(activation, limit)
+    rows, E = logits.shape
+    real = E - identity
+    ff = a.shape[1] // (2 * real)
+    if not a.is_contiguous() or a.shape != (rows, 2 * ff * real):
+        raise ValueError("moe_gated_activate_scored: operands do not fit")
+    out = torch.empty(rows, real * ff, dtype=a.dtype, device=a.device)
+    rest = torch.empty(rows, dtype=torch.float32, device=a.device) if identity else None
+    sums = (_ptr(scaled.sumsq), c_int(scaled.tiles), c_int(scaled.stride), c_int(scaled.shape[1]), c_float(scaled.eps)) \
+        if scaled is not None else (c_void_p(0), c_int(0), c_int(0), c_int(0), c_float(0.0))
+    lib = _latent_moe()
+    _check(lib, lib.ts_moe_gated_activate_scored(
+        c_int(_dt(a)), _ptr(a), c_int(rows), c_int(E), c_int(ff), _ptr(out), c_int(code), c_float(limit), _ptr(logits),
+        _ptr(correction), c_int(top), c_int(groups), c_int(keep), c_int(1 if softmax else 0), c_int(1 if renormalize else 0),
+        c_int(identity), _ptr(rest), *sums, _stream()))
+    return out, rest
 
 
 def moe_gated_activate(a, gates, num_experts, activation="silu", limit=0.0, logits=None, top=0, renormalize=False,
@@ -1954,4 +2018,236 @@ def moe_gated_activate(a, gates, num_experts, activation="silu", limit=0.0, logi
     _check(lib, lib.ts_moe_gated_activate(c_int(_dt(a)), _ptr(a), _ptr(gates), c_int(rows), c_int(num_experts), c_int(ff),
                                           _ptr(out), c_int(code), c_float(limit), _ptr(logits), _ptr(bias), c_int(top),
                                           c_int(1 if renormalize else 0), _stream()))
+    return out
+
+
+# ----------------------------------------------------------------------------- two branches on one stream
+class RowsAdded:
+    """A sub-layer's output to which a multiple of the sub-layer's own input still has to be added:
+    x + factor[t] * rows[t] (the experts whose output is their input).  ``x`` is a tensor or an unfinished
+    product; ``rows`` [T, n] of the compute type; ``factor`` float32 [T].  The kernel that adds it to the
+    32-bit stream adds both; ``materialize()`` gives the sum to any other consumer."""
+
+    def __init__(self, x, factor, rows):
+        self.x, self.factor, self.rows = x, factor, rows
+        self.shape, self.dtype, self.device = tuple(x.shape), x.dtype, x.device
+
+    def materialize(self):
+        x = materialize(self.x)
+        _cuda(x, self.factor, self.rows)
+        out = torch.empty_like(x)
+        lib = _elementwise()
+        _check(lib, lib.ts_add_rows(c_int(_dt(x)), _ptr(x), _ptr(self.factor), _ptr(self.rows), _ptr(out), c_int(x.shape[0]),
+                                    c_int(x.shape[1]), _stream()))
+        return out
+
+
+class BranchSum:
+    """The outputs of a block's branches (mixer, feed-forward) as they are: tensors, unfinished products,
+    a RowsAdded.  ``branch_norm`` adds them to the 32-bit residual; for a few tokens both branches' output
+    products are then one launch.  ``b`` may be None."""
+
+    def __init__(self, a, b=None):
+        self.a, self.b = a, b
+        self.shape, self.dtype, self.device = tuple(a.shape), a.dtype, a.device
+
+    def materialize(self):
+        return PairSum(materialize(self.a), materialize(self.b)).materialize()
+
+
+def _chain(products, out=True, splits=1, residual=None, weights=(None, None), eps=0.0, rest=None):
+    """One launch of one or two PendingProducts whose results add up (csrc/gemm_tcgen05.cu, "chained").
+    With ``residual``: residual += sum (+ bias + rest), returns the ScaledRows of the new residual for each
+    norm weight; else the sum, or with ``out`` False its SplitPartials."""
+    first, second = products[0], products[1] if len(products) > 1 else None
+    M, N = first.shape
+    biases = [p.bias for p in products if p.bias is not None]
+    if len(biases) > 1:
+        raise ValueError("chained products: one of them may have a bias")
+    bias = biases[0] if biases else None
+    device = first.device
+    partials = counters = y = hp1 = hp2 = sumsq = None
+    lib = _gemm_tcgen05()
+    lib.ts_gemm_tcgen05_scratch.restype = c_longlong
+    if residual is not None:
+        hp1 = torch.empty(M, N, dtype=torch.bfloat16, device=device)
+        hp2 = torch.empty(M, N, dtype=torch.bfloat16, device=device) if weights[1] is not None else None
+        sumsq = torch.empty(-(-N // 128), 16, dtype=torch.float32, device=device)
+    else:
+        y = torch.empty(M, N, dtype=torch.bfloat16, device=device) if out else None
+        if splits > 1:
+            partials = torch.empty(lib.ts_gemm_tcgen05_scratch(c_int(M), c_int(N), c_int(splits)), dtype=torch.float32, device=device)
+            counters = _tile_counters(device) if out else None
+    w1 = weights[0]
+    pair = lambda p: (_ptr(p.x), _ptr(p.weight), c_int(p.x.shape[1]), c_longlong(p.x.stride(0)), c_longlong(p.weight.stride(0)))
+    none = (c_void_p(0), c_void_p(0), c_int(0), c_longlong(0), c_longlong(0))
+    _check(lib, lib.ts_gemm_tcgen05_chain(
+        *pair(first), *(pair(second) if second is not None else none), _ptr(y), c_int(M), c_int(N), c_longlong(N), c_int(0),
+        c_int(splits), _ptr(partials), _ptr(counters), _ptr(bias), c_int(_vec_flag(bias, torch.bfloat16) if bias is not None else 0),
+        _ptr(residual), _ptr(w1), _ptr(weights[1]), c_int(_vec_flag(w1, torch.bfloat16) if w1 is not None else 0), _ptr(hp1),
+        _ptr(hp2), _ptr(sumsq), _ptr(rest.factor if rest is not None else None), _ptr(rest.rows if rest is not None else None),
+        _stream()))
+    if residual is not None:
+        tiles = -(-N // 128)
+        return ScaledRows(hp1, sumsq, tiles, eps), ScaledRows(hp2, sumsq, tiles, eps) if hp2 is not None else None
+    return y if out else SplitPartials(partials, splits, M, N, _tile_t(M), torch.bfloat16)
+
+
+def branch_norm(x, residual, weight1, weight2, eps, out_dtype, rows=None, scaled_ok=False):
+    """residual (float32, in place) += x (None, a BranchSum, or anything ``materialize`` takes); returns
+    (rmsnorm(residual) * weight1, the same with weight2 or None): the inputs of a block's two branches.
+    With ``rows`` (int32) only those rows, and the residual is left as it is.  With ``scaled_ok`` the
+    caller takes ScaledRows as well: for up to FUSED_MAX_TOKENS tokens the branches' output products,
+    the residual add and the multiplication by the norm weights are then one launch."""
+    if weight2 is not None and weight2.dtype != weight1.dtype:
+        raise TypeError("branch_norm: the norm weights differ in dtype")
+    if residual.dtype != torch.float32 or not residual.is_contiguous():
+        raise TypeError("the residual stream is contiguous float32")
+    branches = [b for b in ((x.a, x.b) if isinstance(x, BranchSum) else (x,)) if b is not None]
+    rest = None
+    for i, b in enumerate(branches):
+        if isinstance(b, RowsAdded):
+            if rest is not None:
+                branches[i] = b.materialize()
+            else:
+                rest, branches[i] = b, b.x
+    pending = [b for b in branches if isinstance(b, PendingProduct) and not b.wide]
+    if any(tuple(b.shape) != tuple(residual.shape) for b in branches):
+        raise TypeError("branch_norm: a branch does not have the residual's shape")
+    M, n = residual.shape
+    bias = None
+    parts, tensors = _NO_PARTIALS, []
+    if pending and len(pending) == len(branches) and sum(p.bias is not None for p in pending) <= 1:
+        slices = sum(-(-p.x.shape[1] // 64) for p in pending)
+        splits = gemm_splits(M, n, 64 * slices, partials=True)
+        if scaled_ok and rows is None and out_dtype == torch.bfloat16 and M <= FUSED_MAX_TOKENS:
+            _cuda(residual, weight1, weight2)
+            return _chain(pending, splits=min(splits, FUSED_MAX_SPLITS), residual=residual, weights=(weight1, weight2), eps=eps,
+                          rest=rest)
+        if splits > 1:
+            bias = next((p.bias for p in pending if p.bias is not None), None)
+            parts = _chain([PendingProduct(p.x, p.weight) for p in pending], out=False, splits=splits).args()
+        else:
+            tensors = [_chain(pending)]
+    else:
+        for b in branches:
+            b = b.partials() if isinstance(b, PendingProduct) else b
+            if isinstance(b, SplitPartials) and parts is _NO_PARTIALS:
+                parts = b.args()
+            else:
+                tensors.append(materialize(b))
+    for t in tensors:
+        if t.dtype != out_dtype or not t.is_contiguous():
+            raise TypeError("branch_norm: addends are contiguous and of the compute dtype")
+    _cuda(residual, weight1, weight2, rows, *tensors)
+    num_out = M if rows is None else rows.shape[0]
+    out1 = torch.empty(num_out, n, dtype=out_dtype, device=residual.device)
+    out2 = torch.empty_like(out1) if weight2 is not None else None
+    lib = _elementwise()
+    _check(lib, lib.ts_branch_norm(
+        c_int(_DTYPE[out_dtype]), _ptr(tensors[0] if tensors else None), _ptr(tensors[1] if len(tensors) > 1 else None), *parts,
+        _ptr(bias), c_int(_vec_flag(bias, out_dtype) if bias is not None else 0), _ptr(rest.factor if rest is not None else None),
+        _ptr(rest.rows if rest is not None else None), _ptr(residual), _ptr(weight1), _ptr(weight2), c_int(_vec_flag(weight1, out_dtype)),
+        c_float(eps), _ptr(out1), _ptr(out2), _ptr(rows), c_int(num_out), c_int(n), c_int(0 if rows is not None else 1), _stream()))
+    return out1, out2
+
+
+class InputProduct:
+    """A product a part starts with, described so that a block of two branches can run its parts' input
+    products in one launch: h @ weight^T (+ bias), in the compute type or 32-bit."""
+
+    def __init__(self, weight, bias=None, out_float32=False):
+        self.weight, self.bias, self.out_float32 = weight, bias, out_float32
+
+
+BESIDE_MAX_PRODUCTS = 3
+
+
+def linear_beside(groups):
+    """``groups``: (h, [InputProduct, ...]) per branch; returns a list of results per branch.  Up to
+    TCGEN05_MAX_TOKENS bfloat16 rows (up to FUSED_MAX_TOKENS where the h are ScaledRows of one residual) and
+    BESIDE_MAX_PRODUCTS products of one K are one launch; otherwise each runs by itself."""
+    flat = [(h, p) for h, products in groups for p in products]
+    rows = [h.data if isinstance(h, ScaledRows) else h for h, _ in flat]
+    scaled = [h for h, _ in flat if isinstance(h, ScaledRows)]
+    M, K = rows[0].shape
+    one = (1 < len(flat) <= BESIDE_MAX_PRODUCTS and M <= TCGEN05_MAX_TOKENS
+           and all(r.dtype == torch.bfloat16 and tuple(r.shape) == (M, K) and _tcgen05_ok(r, p.weight) for r, (_, p) in zip(rows, flat))
+           and (not scaled or (len(scaled) == len(flat) and M <= FUSED_MAX_TOKENS
+                               and all(h.sumsq is scaled[0].sumsq and h.eps == scaled[0].eps for h in scaled))))
+    if not one:
+        return [[linear(h, p.weight, p.bias, out_float32=p.out_float32) for p in products] for h, products in groups]
+    _cuda(*rows, *[p.weight for _, p in flat], *[p.bias for _, p in flat])
+    outs = [torch.empty(M, p.weight.shape[0], dtype=torch.float32 if p.out_float32 else torch.bfloat16, device=rows[0].device)
+            for _, p in flat]
+    lib = _gemm_tcgen05()
+    lib.ts_gemm_tcgen05_scratch.restype = c_longlong
+    padded = sum(-(-p.weight.shape[0] // 128) for _, p in flat) * 128
+    splits = gemm_splits(M, padded, K)
+    partials = counters = None
+    if splits > 1:
+        partials = torch.empty(lib.ts_gemm_tcgen05_scratch(c_int(M), c_int(padded), c_int(splits)), dtype=torch.float32,
+                               device=rows[0].device)
+        counters = _tile_counters(rows[0].device)
+    n = len(flat)
+    ptrs = lambda ts: (c_void_p * n)(*[t.data_ptr() if t is not None else None for t in ts])
+    ints = lambda vs: (c_int * n)(*vs)
+    longs = lambda vs: (c_longlong * n)(*vs)
+    _check(lib, lib.ts_gemm_tcgen05_beside(
+        c_int(n), ptrs(rows), ptrs([p.weight for _, p in flat]), ptrs(outs), ints([p.weight.shape[0] for _, p in flat]),
+        longs([r.stride(0) for r in rows]), longs([p.weight.stride(0) for _, p in flat]), longs([o.stride(0) for o in outs]),
+        ints([1 if p.out_float32 else 0 for _, p in flat]), ptrs([p.bias for _, p in flat]),
+        ints([_vec_flag(p.bias, torch.bfloat16) if p.bias is not None else 0 for _, p in flat]), c_int(M), c_int(K), c_int(splits),
+        _ptr(partials), _ptr(counters), *(scaled[0].args() if scaled else _NO_SCALE), _stream()))
+    results, at = [], 0
+    for _, products in groups:
+        results.append(outs[at:at + len(products)])
+        at += len(products)
+    return results
+
+
+# ----------------------------------------------------------------------------- a polynomial of normed powers
+def poly_norm(z, coefficients, eps):
+    """[rows, n]: c0 N(z) + c1 N(z^2) + c2 N(z^3) + c3 with powers element by element and
+    N(y) = y / sqrt(mean(y^2) + eps) over the row; ``coefficients`` [4].  32-bit arithmetic."""
+    z = materialize(z)
+    _cuda(z, coefficients)
+    if not z.is_contiguous() or coefficients.shape != (4,):
+        raise TypeError("poly_norm: contiguous rows and four coefficients")
+    out = torch.empty_like(z)
+    lib = _elementwise()
+    _check(lib, lib.ts_poly_norm(c_int(_dt(z)), _ptr(z), _ptr(out), _ptr(coefficients), c_int(_f32(coefficients)), c_float(eps),
+                                 c_int(z.shape[0]), c_int(z.shape[1]), _stream()))
+    return out
+
+
+# ----------------------------------------------------------------------------- convolved heads
+def conv_heads_kvwrite(x, ctx, num_heads, num_kv_heads, dim, vdim, stored_dim, weight=None, state=None, factor=None,
+                       k_cache=None, v_cache=None, slot_mapping=None, page_size=0):
+    """The rows x [T, H dim | G dim | G vdim] of a fused q/k/v projection through a causal convolution over
+    time on every channel (``weight`` [channels, taps], ``state`` float32 [slots, taps - 1, channels] as for
+    ``causal_conv``; None: as they are): returns the query rows [T, H, stored_dim], head h times factor[h]
+    (``factor`` [H] or None), and writes keys and values to the cache slots of ``slot_mapping``, heads
+    padded with zeros.  Without ``slot_mapping`` x holds the queries' columns only."""
+    G = num_kv_heads if slot_mapping is not None else 0
+    channels = num_heads * dim + G * (dim + vdim)
+    taps = weight.shape[1] if weight is not None else 1
+    _cuda(x, weight, state, factor, k_cache, v_cache, slot_mapping)
+    if x.shape[1] != channels or x.stride(1) != 1 or (weight is not None and (weight.shape[0] != channels or not weight.is_contiguous())):
+        raise ValueError("conv_heads_kvwrite: the projection and the convolution do not have heads x size channels")
+    if not 1 <= taps <= CAUSAL_CONV_MAX_TAPS:
+        raise ValueError(f"conv_heads_kvwrite: 1 to {CAUSAL_CONV_MAX_TAPS} taps, got {taps}")
+    if taps > 1 and (state is None or state.dtype != torch.float32 or tuple(state.shape[1:]) != (taps - 1, channels) or not state.is_contiguous()):
+        raise TypeError("conv_heads_kvwrite: the state is contiguous float32 [slots, taps - 1, channels]")
+    if G and (k_cache.dtype != x.dtype or v_cache.dtype != x.dtype or k_cache.shape[-1] != stored_dim or v_cache.shape[-1] != stored_dim
+              or k_cache.shape[1] != G or v_cache.shape[1] != G or not k_cache.is_contiguous() or not v_cache.is_contiguous()):
+        raise TypeError("conv_heads_kvwrite: the cache does not fit the activations")
+    T = x.shape[0]
+    out = torch.empty(T, num_heads, stored_dim, dtype=x.dtype, device=x.device)
+    lib = _sequence()
+    _check(lib, lib.ts_conv_heads_kvwrite(
+        c_int(_f32(x)), _ptr(x), c_longlong(x.stride(0)), _ptr(weight), c_int(_f32(weight) if weight is not None else 0), c_int(taps),
+        _ptr(factor), c_int(_f32(factor) if factor is not None else 0), _ptr(state), _ptr(ctx.state_slots), _ptr(ctx.fresh),
+        _ptr(ctx.cu_q), c_int(ctx.num_requests), c_int(max(1, min(ctx.max_q_len or T, T))), c_int(num_heads), c_int(G), c_int(dim),
+        c_int(vdim), c_int(stored_dim), _ptr(out), _ptr(k_cache), _ptr(v_cache), _ptr(slot_mapping), c_int(page_size), _stream()))
     return out

@@ -29,6 +29,15 @@ element, before the output projection).  Biases on q, k and v go with all of the
 
 ``softcap`` c > 0: the scaled score s becomes c tanh(s / c) before the softmax.
 
+``conv_taps`` n > 0: q, k and v pass a causal convolution over time on every channel directly after
+their projection (the last n - 1 projected rows of a request are its state); ``query_factor``: a
+learned number per query head multiplies its scores (the query row is multiplied, in 32-bit);
+``sink_score``: a sink (as ``sinks``) whose score is this constant for every head; ``value_rotation``
+(a rotary encoding in neighbouring pairs over the whole value): values are turned to their token's
+position before they are cached, and every output row is turned back by its query's position, inside
+the attention kernels; ``borrows_kv``: the layer has no keys and values of its own and reads another
+layer's cache (its run-order entry names it and does not write).
+
 ``differential`` = {"diff": d, "eps": e}: every head has two score maps over the same values.  q
 holds 2 dim columns per head and k 2 dim per key/value head, [map 1 | map 2]; each map is normed
 (``qk_norm``), rotated, capped and softmaxed on its own and gives an output a_1, a_2 over the
@@ -40,12 +49,12 @@ head i reads value head i / 2); ``ops.map_difference`` then combines the pairs."
 from __future__ import annotations
 
 from ..kernels import ops
-from .base import (CacheSpec, Mixer, ParamSpec, Source, build_norm, build_position_encoding,
+from .base import (CacheSpec, Mixer, ParamSpec, Source, StateSpec, build_norm, build_position_encoding,
                    register_mixer)
 
 
 DEFAULT_NAMES = {"q": "q_proj", "k": "k_proj", "v": "v_proj", "o": "o_proj", "q_norm": "q_norm", "k_norm": "k_norm",
-                 "gate": "g_proj", "sinks": "sinks", "lambda_q1": "lq1", "lambda_k1": "lk1", "lambda_q2": "lq2",
+                 "gate": "g_proj", "sinks": "sinks", "query_factor": "q_factor", "conv": "{name}.conv", "lambda_q1": "lq1", "lambda_k1": "lk1", "lambda_q2": "lq2",
                  "lambda_k2": "lk2"}
 
 
@@ -56,7 +65,8 @@ class Attention(Mixer):
     def __init__(self, hidden_size, num_heads, num_kv_heads, head_dim, bias=False, qk_norm=None,
                  position=None, window=0, scale=None, names=None, value_dim=None, unit_norm_eps=None,
                  head_gate=False, keep_first=0, joint_norm=False, norm_eps=0.0, chunk=0, distance_slopes=None,
-                 sinks=False, out_gate=False, softcap=0.0, differential=None):
+                 sinks=False, out_gate=False, softcap=0.0, differential=None, conv_taps=0, query_factor=False,
+                 sink_score=None, value_rotation=None, borrows_kv=False):
         super().__init__()
         self.names = dict(DEFAULT_NAMES, **(names or {}))
         if num_heads % num_kv_heads:
@@ -92,7 +102,24 @@ class Attention(Mixer):
         self.maps = 2 if self.differential else 1
         if self.differential and (extended or self.head_gate or self.unit_norm_eps is not None or bias):
             raise ValueError("attention: two score maps come with a per-head q/k norm, rotation, a window and a soft cap only")
-        self.general = (self.value_dim != head_dim or self.unit_norm_eps is not None or self.head_gate
+        # forms that any of the kernels between projection and attention may be asked for
+        self.conv_taps, self.query_factor, self.borrows_kv = int(conv_taps or 0), bool(query_factor), bool(borrows_kv)
+        self.value_rotation = build_position_encoding(value_rotation) if value_rotation is not None else None
+        self.sink_score = None if sink_score is None else float(sink_score)
+        if not 0 <= self.conv_taps <= ops.CAUSAL_CONV_MAX_TAPS:
+            raise ValueError(f"attention: a convolution of 1 to {ops.CAUSAL_CONV_MAX_TAPS} taps, got {conv_taps}")
+        self.convolved = self.conv_taps > 0 or self.query_factor
+        further = self.convolved or self.borrows_kv or self.value_rotation is not None or self.sink_score is not None
+        if self.convolved and (self.joint_norm or position is not None or qk_norm is not None or unit_norm_eps is not None
+                               or self.value_rotation is not None or self.differential or bias):
+            raise ValueError("attention: a convolution and a factor per query head come without norms, rotation, biases and a second map")
+        if self.value_rotation is not None and (self.value_rotation.rotary_dim != self.value_dim or not self.value_rotation.interleaved
+                                                or self.joint_norm or self.differential or extended):
+            raise ValueError("attention: values turn over their whole size in neighbouring pairs, without a joint norm, chunks, "
+                             "slopes, learned sinks, output gate or a second map")
+        if further and (self.differential or (self.has_sinks and self.sink_score is not None)):
+            raise ValueError("attention: two score maps come alone, and a sink is learned or constant")
+        self.general = (further or self.value_dim != head_dim or self.unit_norm_eps is not None or self.head_gate
                         or self.keep_first > 0 or extended or self.softcap > 0 or self.maps > 1)
         if self.general and ((qk_norm is not None and (extended or self.unit_norm_eps is not None))
                              or (bias and not extended)):
@@ -107,6 +134,8 @@ class Attention(Mixer):
         self.q_size = num_heads * self.maps * head_dim
         self.kv_size = num_kv_heads * self.maps * head_dim
         self.v_size = num_kv_heads * self.value_dim
+        if self.borrows_kv:
+            self.kv_size = self.v_size = 0
         self.map_factor = None       # lambda of the two maps, made when the tensors are bound
         self.gate_size = num_heads if self.head_gate else (num_heads * self.value_dim if self.out_gate else 0)
 
@@ -116,12 +145,17 @@ class Attention(Mixer):
             out[self.names["q_norm"]], out[self.names["k_norm"]] = self.q_norm, self.k_norm
         if self.position is not None:
             out["position"] = self.position
+        if self.value_rotation is not None:
+            out["value_rotation"] = self.value_rotation
         return out
 
     def param_specs(self):
         q, kv, vs = self.q_size, self.kv_size, self.v_size
         nm = self.names
         rows = ((nm["q"], 0, q), (nm["k"], q, q + kv), (nm["v"], q + kv, q + kv + vs))
+        if self.borrows_kv:
+            rows = rows[:1]
+        qkv_rows = rows
         if self.gate_size:
             rows += ((nm["gate"], q + kv + vs, q + kv + vs + self.gate_size),)
         specs = {
@@ -134,12 +168,18 @@ class Attention(Mixer):
             # drawn like a matrix in the random-weights mode: a bias of zeros would hide a fault
             # (the gate's rows, where there are any, have no bias: ``bind`` zeroes theirs)
             specs["qkv_proj.bias"] = ParamSpec((q + kv + vs + self.gate_size,), role="matrix", init="normal", sources=tuple(
-                Source(f"{n}.bias", a, b) for n, a, b in rows[:3]))
+                Source(f"{n}.bias", a, b) for n, a, b in qkv_rows))
         if self.joint_norm:
             specs["q_norm.weight"] = ParamSpec((q,), role="vector", init="norm_weight",
                                                sources=(Source(f"{nm['q_norm']}.weight", 0, q),))
             specs["k_norm.weight"] = ParamSpec((kv,), role="vector", init="norm_weight",
                                                sources=(Source(f"{nm['k_norm']}.weight", 0, kv),))
+        if self.conv_taps:
+            specs["qkv_conv.weight"] = ParamSpec((q + kv + vs, self.conv_taps), init="wide", sources=tuple(
+                Source(nm["conv"].format(name=n) + ".weight", a, b) for n, a, b in qkv_rows))
+        if self.query_factor:
+            specs["query_factor"] = ParamSpec((self.num_heads,), role="vector", init="unit_interval",
+                                              sources=(Source(nm["query_factor"], 0, self.num_heads),))
         if self.has_sinks:
             specs["sinks"] = ParamSpec((self.num_heads,), role="vector", init="wide", sources=(Source(nm["sinks"], 0, self.num_heads),))
         if self.differential:
@@ -163,6 +203,9 @@ class Attention(Mixer):
 
     def prepare(self, runtime):
         super().prepare(runtime)
+        if self.sink_score is not None:
+            import torch
+            self.sinks = torch.full((self.num_heads,), self.sink_score, dtype=torch.float32, device=runtime.device)
         if self.slope_values is not None:
             import torch
             self.slopes = torch.tensor(self.slope_values, dtype=torch.float32, device=runtime.device)
@@ -177,6 +220,11 @@ class Attention(Mixer):
                              keep_first=self.keep_first)
         return CacheSpec(kind, self.num_kv_heads, self.stored_dim, self.window, keep_first=self.keep_first)
 
+    def state_spec(self):
+        if self.conv_taps < 2:
+            return None
+        return StateSpec((self.conv_taps - 1, self.q_size + self.kv_size + self.v_size), "float32")
+
     def _biased(self):
         return self.chunk > 0 or self.slope_values is not None
 
@@ -186,47 +234,61 @@ class Attention(Mixer):
         return ops.prefill_tile_queries(dtype, self.num_heads * self.maps, self.num_kv_heads * self.maps, self.stored_dim,
                                         page_size)
 
-    def _forward_general(self, h, ctx, call):
-        qkv = ops.materialize(ops.linear(h, self.w["qkv_proj.weight"], self.w.get("qkv_proj.bias")))
+    def input_products(self):
+        """The product this mixer starts with (the general form), for a block that runs it beside others."""
+        return [ops.InputProduct(self.w["qkv_proj.weight"], self.w.get("qkv_proj.bias"))] if self.general else None
+
+    def _query_rows(self, qkv, ctx, call, cache, view):
+        """The attention kernels' query rows [T, heads, stored_dim] of this step's projected rows; keys and
+        values go to the cache on the way."""
         q_end, k_end = self.q_size, self.q_size + self.kv_size
         v_end = k_end + self.v_size
-        cache = ctx.cache(call.cache)
-        view = ctx.group(cache.group)
-        if self.joint_norm or self._biased() or self.has_sinks or self.out_gate:
-            q = ops.joint_norm_kvwrite(
-                qkv[:, :q_end], qkv[:, q_end:k_end], qkv[:, k_end:v_end], self.num_heads, self.num_kv_heads, self.head_dim,
+        slots = view.slot_mapping if call.writes_cache and not self.borrows_kv else None
+        k, v = (None, None) if self.borrows_kv else (qkv[:, q_end:k_end], qkv[:, k_end:v_end])
+        if self.convolved:
+            return ops.conv_heads_kvwrite(
+                qkv[:, :v_end], ctx, self.num_heads, self.num_kv_heads, self.head_dim, self.value_dim, self.stored_dim,
+                weight=self.w.get("qkv_conv.weight"), state=ctx.state(call.state) if self.conv_taps > 1 else None,
+                factor=self.w.get("query_factor"), k_cache=cache.k, v_cache=cache.v, slot_mapping=slots, page_size=view.page_size)
+        if (self.joint_norm or self._biased() or self.has_sinks or self.out_gate) and not self.borrows_kv:
+            return ops.joint_norm_kvwrite(
+                qkv[:, :q_end], k, v, self.num_heads, self.num_kv_heads, self.head_dim,
                 self.value_dim, self.stored_dim, self.w.get("q_norm.weight"), self.w.get("k_norm.weight"), self.norm_eps,
-                k_cache=cache.k, v_cache=cache.v, slot_mapping=view.slot_mapping if call.writes_cache else None,
-                page_size=view.page_size)
-            out = ops.paged_attention(q, cache.k, cache.v, view, ctx, self.scale, self.window, keep_first=self.keep_first,
-                                      sinks=self.w.get("sinks"), chunk=self.chunk, slopes=self.slopes)
-            if self.out_gate:
-                out = ops.gate_columns(out, qkv[:, v_end:], self.value_dim)
-            elif self.head_gate or self.stored_dim != self.value_dim:
-                out = ops.head_gate(out, qkv[:, v_end:] if self.head_gate else None, self.value_dim)
-            else:
-                out = out.view(out.shape[0], self.num_heads * self.value_dim)
-            return ops.linear(out, self.w["o_proj.weight"], allow_pending=True)
+                k_cache=cache.k, v_cache=cache.v, slot_mapping=slots, page_size=view.page_size)
         M = self.maps
-        q = ops.rope_unit_kvwrite(
-            qkv[:, :q_end], qkv[:, q_end:k_end], qkv[:, k_end:v_end], ctx.positions, self.num_heads * M,
+        return ops.rope_unit_kvwrite(
+            qkv[:, :q_end], k, v, ctx.positions, self.num_heads * M,
             self.num_kv_heads * M, self.head_dim, self.value_dim, self.stored_dim, rotary=self.position,
             unit_norm=self.unit_norm_eps is not None, eps=self.unit_norm_eps or 0.0, k_cache=cache.k, v_cache=cache.v,
-            slot_mapping=view.slot_mapping if call.writes_cache else None, page_size=view.page_size,
+            slot_mapping=slots, page_size=view.page_size,
             q_weight=self.q_norm.w["weight"] if self.q_norm is not None else None,
             k_weight=self.k_norm.w["weight"] if self.k_norm is not None else None,
-            pre_eps=self.q_norm.eps if self.q_norm is not None else 0.0, maps=M)
+            pre_eps=self.q_norm.eps if self.q_norm is not None else 0.0, maps=M, value_rotary=self.value_rotation)
+
+    def forward_projected(self, projected, h, ctx, call):
+        """What follows the input product(s); ``projected``: their results, in the order of ``input_products``."""
+        qkv = ops.materialize(projected[0])
+        v_end = self.q_size + self.kv_size + self.v_size
+        cache = ctx.cache(call.cache)
+        view = ctx.group(cache.group)
+        q = self._query_rows(qkv, ctx, call, cache, view)
         out = ops.paged_attention(q, cache.k, cache.v, view, ctx, self.scale, self.window, keep_first=self.keep_first,
-                                  softcap=self.softcap)
-        if M > 1:
+                                  sinks=self.w.get("sinks", self.sinks), chunk=self.chunk, slopes=self.slopes, softcap=self.softcap,
+                                  turn=self.value_rotation)
+        if self.maps > 1:
             d = self.differential
             out = ops.map_difference(out, self.num_heads, self.num_kv_heads, self.value_dim, self.map_factor,
                                      float(d["eps"]), 1.0 - float(d["diff"]))
+        elif self.out_gate:
+            out = ops.gate_columns(out, qkv[:, v_end:], self.value_dim)
         elif self.head_gate or self.stored_dim != self.value_dim:
             out = ops.head_gate(out, qkv[:, v_end:] if self.head_gate else None, self.value_dim)
         else:
             out = out.view(out.shape[0], self.num_heads * self.value_dim)
         return ops.linear(out, self.w["o_proj.weight"], allow_pending=True)
+
+    def _forward_general(self, h, ctx, call):
+        return self.forward_projected([ops.linear(h, self.w["qkv_proj.weight"], self.w.get("qkv_proj.bias"))], h, ctx, call)
 
     def forward(self, h, ctx, call):
         if self.general:

@@ -198,6 +198,12 @@ class Mixer(Part):
         function then packs those lists with the step's other inputs."""
         return 0
 
+    def input_products(self):
+        """None, or the products of h this part starts with (``ops.InputProduct``): a block of two branches
+        may then run both branches' products in one launch and call ``forward_projected(results, h,
+        ctx, call)`` (a feed-forward: without ``call``) in place of ``forward``.  h may be a ScaledRows there."""
+        return None
+
     def forward(self, h, ctx, call):
         """h [T, hidden] in the compute dtype -> [T, hidden] (a tensor, or what ops.linear
         returned with allow_partials=True).  ``call`` is the
@@ -209,6 +215,10 @@ class Mixer(Part):
 class FeedForward(Part):
     tree_name = "mlp"
     accepts_scaled_rows = False       # as for a Mixer
+
+    def input_products(self):
+        """As for a Mixer."""
+        return None
 
     def forward(self, h, ctx):
         raise NotImplementedError

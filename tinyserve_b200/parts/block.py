@@ -4,7 +4,7 @@
 (x, residual); each norm first adds x to the residual, then normalises it; the
 sub-layer's output becomes the next x, so that r1 = r0 + mixer(norm1(r0)),
 r2 = r1 + ffn(norm2(r1)).  Another arrangement is another class in ARRANGEMENTS ("parallel": mixer
-and feed-forward side by side on one norm; "sandwich": a norm before and after each sub-layer).
+and feed-forward side by side on one norm; "parallel_two_norms": each on a norm of its own; "sandwich": a norm before and after each sub-layer).
 
 The block also owns what lies below the parts' interfaces: a product may hand its result on
 unfinished (split-K partial tiles, a product that has not run yet, rows without their norm
@@ -130,6 +130,53 @@ class ParallelBlock(Part):
         return ops.PairSum(mixed, self.ffn.forward(h, ctx) if self.ffn is not None else None)
 
 
+class ParallelTwoNormsBlock(Part):
+    """Mixer and feed-forward side by side, each on a norm of its own of the same stream:
+    r <- r + (mixer(norm1(r)) + ffn(norm2(r))).  The two RMS norms share their factor, so one kernel takes
+    in what the block before left and writes both branches' inputs (``ops.branch_norm``).  For a few
+    tokens both branches' input products are one launch (``ops.linear_beside``), and both output
+    products with the residual add and the next block's norm weights another one; what a branch returns
+    travels on as it is (``ops.BranchSum``).  A layer without a feed-forward (``LayerSpec.ffn`` None) is
+    r + mixer(norm1(r))."""
+    capturable = True
+
+    def __init__(self, spec: LayerSpec, hidden_size: int):
+        super().__init__()
+        self.mixer = build_mixer(spec.mixer)
+        self.ffn = build_feed_forward(spec.ffn) if spec.ffn is not None else None
+        self.input_norm = build_norm(spec.norm, hidden_size)
+        self.ffn_norm = build_norm(spec.norm, hidden_size) if self.ffn is not None else None
+        for norm in (self.input_norm, self.ffn_norm):
+            if norm is not None and not hasattr(norm, "eps"):
+                raise ValueError("parallel block of two norms: its norms are RMS norms")
+        self._names = {"mixer": spec.name_of("mixer", self.mixer.tree_name),
+                       "ffn": spec.name_of("ffn", self.ffn.tree_name if self.ffn is not None else ""),
+                       "input_norm": spec.name_of("input_norm"), "ffn_norm": spec.name_of("ffn_norm", "ffn_norm")}
+
+    def children(self):
+        n = self._names
+        out = {n["mixer"]: self.mixer, n["input_norm"]: self.input_norm}
+        if self.ffn is not None:
+            out.update({n["ffn"]: self.ffn, n["ffn_norm"]: self.ffn_norm})
+        return out
+
+    def forward(self, x, residual, ctx, call):
+        (w1, eps), w2 = self.input_norm.rms_parameters(), None
+        if self.ffn is not None:
+            w2 = self.ffn_norm.rms_parameters()[0]
+        mixer_in = self.mixer.input_products()
+        ffn_in = self.ffn.input_products() if self.ffn is not None else []
+        beside = mixer_in is not None and ffn_in is not None
+        h1, h2 = ops.branch_norm(x, residual, w1, w2, eps, ctx.dtype, scaled_ok=beside)
+        if residual.shape[0] > ops.TCGEN05_MAX_TOKENS or not beside:
+            # (many tokens: library products; a part decides for itself how it runs them)
+            mixed = self.mixer.forward(h1, ctx, call)
+            return ops.BranchSum(mixed, self.ffn.forward(h2, ctx) if self.ffn is not None else None)
+        projected = ops.linear_beside([(h1, mixer_in)] + ([(h2, ffn_in)] if self.ffn is not None else []))
+        mixed = self.mixer.forward_projected(projected[0], h1, ctx, call)
+        return ops.BranchSum(mixed, self.ffn.forward_projected(projected[1], h2, ctx) if self.ffn is not None else None)
+
+
 class SandwichBlock(Part):
     """A norm before and after each sub-layer: r <- r + post1(mixer(pre1(r))), then
     r <- r + post2(ffn(pre2(r))).  What a sub-layer returns travels on with its post-norm
@@ -239,7 +286,7 @@ class PostNormBlock(Part):
         return None
 
 
-ARRANGEMENTS = {"pre_norm": PreNormBlock, "parallel": ParallelBlock, "sandwich": SandwichBlock,
+ARRANGEMENTS = {"pre_norm": PreNormBlock, "parallel": ParallelBlock, "parallel_two_norms": ParallelTwoNormsBlock, "sandwich": SandwichBlock,
                 "post_norm": PostNormBlock}
 
 

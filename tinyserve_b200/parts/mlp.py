@@ -4,6 +4,10 @@ then the matching up rows (when the width allows), so that a 128-row tile of the
 holds both and can apply the activation in its epilogue; the activation kernel reads the same
 layout where the product is someone else's.
 
+``PolyNormMLP`` is a feed-forward without a gate: down(act(up(x))), both with biases, where act is a
+polynomial of normed powers, c0 N(z) + c1 N(z^2) + c2 N(z^3) + c3 with four learned numbers and N(y) =
+y / sqrt(mean(y^2) + eps) over a token's whole row (``ops.poly_norm``).
+
 ``activation`` "bounded_swish" with ``limit`` L: g = min(gate(x), L), u = clamp(up(x), -L, L),
 down(g sigmoid(1.702 g) (u + 1))."""
 from __future__ import annotations
@@ -45,3 +49,38 @@ class GatedMLP(FeedForward):
 
 
 register_feed_forward("gated_mlp", GatedMLP)
+
+
+class PolyNormMLP(FeedForward):
+    tree_name = "mlp"
+    capturable = True
+    accepts_scaled_rows = True
+
+    def __init__(self, hidden_size, intermediate_size, eps, names=None):
+        super().__init__()
+        self.names = dict(DEFAULT_NAMES, **dict({"act": "act"}, **(names or {})))
+        self.hidden_size, self.intermediate_size, self.eps = hidden_size, intermediate_size, float(eps)
+
+    def param_specs(self):
+        i, n, nm = self.intermediate_size, self.hidden_size, self.names
+        # (the biases and coefficients drawn so that losing one shows in the random-weights mode)
+        return {
+            "up_proj.weight": ParamSpec((i, n), sources=(Source(f"{nm['up']}.weight", 0, i),)),
+            "up_proj.bias": ParamSpec((i,), role="vector", init="around_zero", sources=(Source(f"{nm['up']}.bias", 0, i),)),
+            "down_proj.weight": ParamSpec((n, i), sources=(Source(f"{nm['down']}.weight", 0, n),)),
+            "down_proj.bias": ParamSpec((n,), role="vector", init="around_zero", sources=(Source(f"{nm['down']}.bias", 0, n),)),
+            "act": ParamSpec((4,), role="vector", init="wide", sources=(Source(nm["act"], 0, 4),)),
+        }
+
+    def input_products(self):
+        return [ops.InputProduct(self.w["up_proj.weight"], self.w["up_proj.bias"])]
+
+    def forward_projected(self, projected, h, ctx):
+        act = ops.poly_norm(projected[0], self.w["act"], self.eps)
+        return ops.linear(act, self.w["down_proj.weight"], self.w["down_proj.bias"], allow_pending=True)
+
+    def forward(self, h, ctx):
+        return self.forward_projected([ops.linear(h, p.weight, p.bias) for p in self.input_products()], h, ctx)
+
+
+register_feed_forward("poly_norm_mlp", PolyNormMLP)

@@ -185,8 +185,8 @@ class DecoderModel(Part):
         hidden = add_and_norm(self.norm, x, residual, rows=ctx.logit_rows, compute_dtype=ctx.dtype)
         head = self.lm_head.w["weight"] if self.lm_head is not None else self.embed_tokens.w["weight"]
         logits = ops.linear(hidden, head, out_float32=True)
-        if self.spec.logit_softcap > 0:
-            ops.softcap_(logits, self.spec.logit_softcap)
+        if self.spec.logit_softcap > 0 or self.spec.logit_scale != 1.0:
+            ops.softcap_(logits, self.spec.logit_softcap, self.spec.logit_scale)
         return logits
 
 
