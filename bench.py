@@ -29,6 +29,12 @@ kept first tokens, a mixture of experts whose active weights equal Qwen3's feed-
 
 measures Babadra (latent attention, attention with two capped score maps per head, bounded gated
 feed-forwards, dense and as experts, a repeated group of layers) beside Delilorn, the closest design.
+
+    python bench.py --arch gunulorn [--sizes 2048,4096]
+
+measures Gunulorn (mixer and feed-forward side by side on two norms, convolved attention, window attention
+over turned values, a polynomial of normed powers, experts beside identity experts) beside Babadra, the
+closest design (dense and gated-expert feed-forwards in turn, grouped-query attention).
 """
 from __future__ import annotations
 
@@ -433,6 +439,26 @@ def babadra_shapes(width):
                "embedding": {"scale": float(width) ** 0.5}, "logit_softcap": 30.0, "loop": {"start": 1, "stop": 3, "times": 2},
                "layers": order + order}
     return babadra, delilorn
+
+
+def gunulorn_shapes(width):
+    """A Gunulorn of real layer sizes at ``width``: convolved attention with a dense feed-forward, window
+    attention (1,024 keys beside 4 kept tokens) over turned values with experts, three times; the second
+    and third convolved layers read the first one's keys and values: six blocks.  As many query heads of
+    128 as the Delilorn of the same width, 8 gated experts and 2 identity experts of which a token takes
+    2; dense and expert feed-forwards hold as many weights as those of the Babadra beside it."""
+    babadra, delilorn = babadra_shapes(width)
+    heads, vocab = width // 128, 32768
+    ff, ffe = babadra["layers"][0]["mlp"]["ff"] * 3 // 2, babadra["layers"][1]["mlp"]["expert"]["ff"]
+    window = delilorn["layers"][3]["mixer"]
+    base = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5}
+    conv, dense = dict(base, conv=4), {"kind": "dense", "ff": ff}
+    turned = {"type": "attention_2", "mixer": dict(base, rot={"base": 2.5e5, "dims": 64}, mask=window["mask"]),
+              "mlp": {"kind": "moe", "expert": {"ff": ffe}, "router": {"experts": 8, "identity": 2, "top": 2}}}
+    reader = {"type": "attention", "mixer": dict(conv, kv_from=0), "mlp": dense}
+    gunulorn = {"architecture": "Gunulorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_scale": 0.5,
+                "logit_softcap": 30.0, "layers": [{"type": "attention", "mixer": conv, "mlp": dense}, turned, reader, turned, reader, turned]}
+    return gunulorn, babadra
 
 
 def _time_us(fn, iters=20):
@@ -922,16 +948,160 @@ def babadra_kernel_table(width, peaks):
     return out
 
 
+def gunulorn_kernel_table(width, peaks):
+    """Gunulorn's kernels beside the like kernels of Babadra, Delilorn and Tarivik at this width, time over
+    roofline time.  Attention with a sink beside plain attention of as many heads; window attention over
+    turned values beside Delilorn's window attention (prefill: FLOPs of the visible keys over the library's
+    GEMM rate; decode: bytes of the cached keys and values); the convolution of q, k, v with the cache write
+    beside Tarivik's convolution of as many channels; rotation of q, k and values with the cache write beside
+    Delilorn's rotation and cache write (bytes in and out); the experts and the dense feed-forward beside
+    Babadra's (prefill: FLOPs; decode: bytes of the weights); the polynomial of normed powers beside the
+    gated activation (bytes); what two branches leave, added and normed twice, beside Delilorn's norm + add +
+    norm (bytes); and for a decode step both branches' input products, and both output products with the
+    residual add, as one launch each beside the launches of one product alone (bytes of the weights).  All
+    launches are replayed from a graph: the host's time between them is not in the figures."""
+    import torch
+    from tinyserve_b200.engine.batch import GroupView, StepContext
+    from tinyserve_b200.kernels import ops
+    from tinyserve_b200.parts.mlp import PolyNormMLP
+    from tinyserve_b200.parts.moe import MixtureOfExperts
+    from tinyserve_b200.parts.rotary import Rotary
+    dev, bf = "cuda:0", torch.bfloat16
+    raw, beside = gunulorn_shapes(width)
+    win, dense, moe = raw["layers"][1]["mixer"], raw["layers"][0]["mlp"], raw["layers"][1]["mlp"]
+    H, G, D = win["heads"], win["kv_heads"], 128
+    out = {}
+    rnd = lambda *s, scale=1.0: (torch.randn(*s, device=dev) * scale).to(bf)
+
+    def frac(key, us, roof):
+        out[key] = {"us": round(us, 1), "roofline_us": round(roof, 2), "frac": round(roof / us, 3)}
+
+    def rotary(dims, interleaved):
+        cos, sin = Rotary.tables(dims, 2.5e5, CONTEXT)
+        return type("R", (), {"cos": cos.to(dev), "sin": sin.to(dev), "rotary_dim": dims, "interleaved": interleaved})()
+
+    for name, lengths, starts in (("prefill_2048", [2048], [0]), ("decode_b8", [1] * 8, [2048] * 8)):
+        T, B = sum(lengths), len(lengths)
+        timed = _time_graph_us
+        moved = lambda bytes_: bytes_ / (peaks["hbm_gbs"] * 1e3)
+        kv_len, page = starts[0] + lengths[0], 64
+        pages_per = -(-kv_len // page)
+        cu = torch.tensor([0] + list(torch.tensor(lengths).cumsum(0)), dtype=torch.int32, device=dev)
+        table = (torch.arange(B * pages_per, dtype=torch.int32, device=dev) + 1).view(B, pages_per)
+        positions = torch.cat([torch.arange(s, s + m) for s, m in zip(starts, lengths)]).int().to(dev)
+        slots = torch.cat([table[b, (s + torch.arange(m, device=dev)) // page] * page + (s + torch.arange(m, device=dev)) % page
+                           for b, (s, m) in enumerate(zip(starts, lengths))]).int()
+        kc, vc = (torch.randn(B * pages_per + 1, G, page, D, device=dev).to(bf) for _ in range(2))
+        sc = StepContext()
+        sc.num_tokens, sc.num_requests, sc.max_q_len, sc.max_kv_len = T, B, max(lengths), kv_len
+        sc.cu_q, sc.kv_lens, sc.positions = cu, torch.full((B,), kv_len, dtype=torch.int32, device=dev), positions
+        sc.state_slots, sc.fresh = torch.arange(B, dtype=torch.int32, device=dev), torch.zeros(B, dtype=torch.int32, device=dev)
+        sc.host = {"cu_q": cu.tolist(), "kv_lens": [kv_len] * B}
+        view = GroupView(page, pages_per, None, table, kc.shape[0])
+        q = rnd(T, H, D)
+
+        def attention(**kw):
+            run = lambda: ops.paged_attention(q, kc, vc, view, sc, D ** -0.5, **kw)
+            run()                                                                     # (work lists)
+            return timed(run)
+
+        def roof(window=0, keep=0):
+            pos = torch.arange(kv_len - lengths[0], kv_len)
+            n = pos + 1 if not window else torch.minimum(pos + 1, torch.full_like(pos, window)) + torch.clamp(
+                torch.minimum(pos + 1 - window, torch.full_like(pos, keep)), min=0)
+            seen = float(n.sum())
+            return 4.0 * H * D * seen / (peaks["bf16_tflops"] * 1e6) if T > B else moved(B * seen * 2 * G * D * 2)
+
+        size, keep = win["mask"]["size"], win["mask"]["keep_first"]
+        frac(f"sink_attention_{name}", attention(sinks=torch.randn(H, device=dev)), roof())
+        frac(f"plain_attention_{name}", attention(), roof())
+        frac(f"turned_window_attention_{name}", attention(window=size, keep_first=keep, sinks=torch.zeros(H, device=dev), turn=rotary(D, True)),
+             roof(size, keep))
+        frac(f"delilorn_window_attention_{name}", attention(window=size, keep_first=keep), roof(size, keep))
+        # what stands before the attention kernels
+        C = (H + 2 * G) * D
+        qkv, w, wt = rnd(T, C), rnd(C, 4), rnd(4, C)
+        state, factor = torch.zeros(B, 3, C, device=dev), rnd(H)
+        frac(f"conv_heads_cache_write_{name}", timed(lambda: ops.conv_heads_kvwrite(
+            qkv, sc, H, G, D, D, D, weight=wt, state=state, factor=factor, k_cache=kc, v_cache=vc, slot_mapping=slots, page_size=page)),
+            moved(T * C * 4))
+        frac(f"tarivik_causal_conv_{name}", timed(lambda: ops.causal_conv(qkv, w, state, sc, bf, activation="silu")), moved(T * C * 4))
+        q_end, k_end = H * D, (H + G) * D
+        rope = lambda rot, values: ops.rope_unit_kvwrite(qkv[:, :q_end], qkv[:, q_end:k_end], qkv[:, k_end:], positions, H, G, D, D, D, rotary=rot,
+                                                         k_cache=kc, v_cache=vc, slot_mapping=slots, page_size=page, value_rotary=values)
+        rot_pairs, rot_half, turn = rotary(64, True), rotary(64, False), rotary(D, True)
+        frac(f"rotary_values_cache_write_{name}", timed(lambda: rope(rot_pairs, turn)), moved(T * C * 4))
+        frac(f"delilorn_rotary_cache_write_{name}", timed(lambda: rope(rot_half, None)), moved(T * C * 4))
+        # feed-forwards
+        E, I, top, ffe, ff = moe["router"]["experts"], moe["router"]["identity"], moe["router"]["top"], moe["expert"]["ff"], dense["ff"]
+        ffb = beside["layers"][0]["mlp"]["ff"]
+        torch.manual_seed(0)
+        mine = MixtureOfExperts(width, ffe, E, top, activation="silu_gated", router="softmax_corrected", identity=I)
+        theirs = MixtureOfExperts(width, ffe, E, top, activation="bounded_swish_gated", router="softmax_chosen", limit=7.0, router_bias=True)
+        up, down = rnd(E * 2 * ffe, width, scale=0.02), rnd(E * width, ffe, scale=0.02)
+        mine.bind({"router.weight": rnd(E + I, width, scale=0.1), "correction": torch.randn(E + I, device=dev) * 0.01, "up.weight": up, "down.weight": down})
+        theirs.bind({"router.weight": rnd(E, width, scale=0.1), "router.bias": torch.randn(E, device=dev), "up.weight": up, "down.weight": down})
+        poly = PolyNormMLP(width, ff, 1e-6)
+        poly.bind({"up_proj.weight": rnd(ff, width, scale=0.02), "up_proj.bias": rnd(ff), "down_proj.weight": rnd(width, ff, scale=0.02),
+                   "down_proj.bias": rnd(width), "act": torch.tensor([0.5, 0.25, -0.5, 0.1], device=dev)})
+        h = rnd(T, width)
+        gate_up, gdown = rnd(2 * ffb, width, scale=0.02), rnd(width, ffb, scale=0.02)
+        block = ops.GATED_BLOCK if ffb % ops.GATED_BLOCK == 0 else 0
+        us_mine = timed(lambda: ops.materialize(mine.forward(h, None)))
+        us_theirs = timed(lambda: ops.materialize(theirs.forward(h, None)))
+        us_poly = timed(lambda: ops.materialize(poly.forward(h, None)))
+        us_dense = timed(lambda: ops.materialize(ops.linear(ops.gated_linear(h, gate_up, "bounded_swish", block, 7.0), gdown)))
+        if T > B:
+            # (of the top choices the share of the real experts is computed)
+            share = float((mine._route(ops.linear(h, mine.w["router.weight"], out_float32=True))[0] > 0).sum()) / (T * top)
+            flops = lambda f: f / (peaks["bf16_tflops"] * 1e6)
+            frac(f"experts_{name}", us_mine, flops(6.0 * T * top * share * width * ffe))
+            out[f"experts_{name}"]["chosen_of_real_experts"] = round(share, 3)
+            frac(f"babadra_experts_{name}", us_theirs, flops(6.0 * T * top * width * ffe))
+            frac(f"poly_feed_forward_{name}", us_poly, flops(4.0 * T * width * ff))
+            frac(f"babadra_feed_forward_{name}", us_dense, flops(6.0 * T * width * ffb))
+        else:
+            frac(f"experts_{name}", us_mine, moved(3.0 * E * width * ffe * 2))
+            frac(f"babadra_experts_{name}", us_theirs, moved(3.0 * E * width * ffe * 2))
+            frac(f"poly_feed_forward_{name}", us_poly, moved(2.0 * width * ff * 2))
+            frac(f"babadra_feed_forward_{name}", us_dense, moved(3.0 * width * ffb * 2))
+        z, z2 = rnd(T, ff), rnd(T, 2 * ff)
+        frac(f"poly_norm_{name}", timed(lambda: ops.poly_norm(z, poly.w["act"], 1e-6)), moved(T * ff * 4))
+        frac(f"gated_activation_{name}", timed(lambda: ops.gated_activation(z2, "silu", ops.GATED_BLOCK)), moved(T * ff * 6))
+        # the stream
+        res, y, y2 = torch.randn(T, width, device=dev), rnd(T, width), rnd(T, width)
+        w1, w2 = torch.ones(width, device=dev), torch.ones(width, device=dev)
+        frac(f"branch_norm_{name}", timed(lambda: ops.branch_norm(ops.BranchSum(y, y2), res, w1, w2, 1e-6, bf)), moved(T * width * (8 + 4 + 4)))
+        frac(f"delilorn_normed_add_rmsnorm_{name}", timed(lambda: ops.normed_add_rmsnorm(ops.NormedAddend(y, w1, 1e-6), res, w1, 1e-6, bf)),
+             moved(T * width * (8 + 2 + 2)))
+        if T == B:
+            wqkv, wo = rnd(C, width, scale=0.02), rnd(width, H * D, scale=0.02)
+            attn, act = rnd(T, H * D), rnd(T, ff)
+            ins = [(h, [ops.InputProduct(wqkv)]), (h, poly.input_products())]
+            frac("input_products_together_decode_b8", timed(lambda: ops.linear_beside(ins)), moved((C + ff) * width * 2))
+            ins_moe = [(h, [ops.InputProduct(wqkv)]), (h, mine.input_products())]
+            frac("input_products_with_experts_decode_b8", timed(lambda: ops.linear_beside(ins_moe)), moved((C + E * 2 * ffe + E + I) * width * 2))
+            frac("one_input_product_decode_b8", timed(lambda: ops.linear(h, poly.w["up_proj.weight"], poly.w["up_proj.bias"])), moved(ff * width * 2))
+            pair = lambda: ops.branch_norm(ops.BranchSum(ops.linear(attn, wo, allow_pending=True),
+                                                         ops.linear(act, poly.w["down_proj.weight"], poly.w["down_proj.bias"], allow_pending=True)),
+                                           res, w1, w2, 1e-6, bf, scaled_ok=True)
+            frac("output_products_and_residual_decode_b8", timed(pair), moved((H * D + ff) * width * 2))
+            frac("one_output_product_and_residual_decode_b8", timed(lambda: ops.add_rmsnorm(
+                ops.linear(act, poly.w["down_proj.weight"], allow_pending=True), res, w1, 1e-6, bf, scaled_ok=True)), moved(ff * width * 2))
+    return out
+
+
 # design -> (its shapes and those of the model beside it, its kernel table, the name of the model beside it)
 ARCH_BENCHES = {"dudatar": (dudatar_shapes, kernel_table, "qwen3"), "delilorn": (delilorn_shapes, delilorn_kernel_table, "qwen3"),
                 "tarivik": (tarivik_shapes, tarivik_kernel_table, "delilorn"),
-                "babadra": (babadra_shapes, babadra_kernel_table, "delilorn")}
+                "babadra": (babadra_shapes, babadra_kernel_table, "delilorn"),
+                "gunulorn": (gunulorn_shapes, gunulorn_kernel_table, "babadra")}
 
 
 def arch_main(a) -> int:
     """``--arch dudatar`` / ``--arch delilorn``: the design beside Qwen3 at equal size; ``--arch tarivik`` and
-    ``--arch babadra``: beside Delilorn, the closest design (experts, latent attention, matrix-state mixers).  One
-    JSON line."""
+    ``--arch babadra``: beside Delilorn, the closest design (experts, latent attention, matrix-state mixers);
+    ``--arch gunulorn``: beside Babadra.  One JSON line."""
     import torch
     from tinyserve_b200 import LLM
     from tinyserve_b200.config import config_from_dict
@@ -1001,10 +1171,10 @@ def main() -> int:
     ap.add_argument("--no-points", action="store_true", help="skip batch 1 / 64 and prefill")
     ap.add_argument("--no-workloads", action="store_true",
                     help="skip the 0.6B burst, the 32B run and the long-context decode")
-    ap.add_argument("--arch", choices=["qwen3", "dudatar", "delilorn", "tarivik", "babadra"], default="qwen3",
+    ap.add_argument("--arch", choices=["qwen3", "dudatar", "delilorn", "tarivik", "babadra", "gunulorn"], default="qwen3",
                     help="dudatar, delilorn: measure that design beside Qwen3 at equal size instead of the default workload; "
-                         "tarivik, babadra: beside Delilorn")
-    ap.add_argument("--sizes", default="2048,4096", help="--arch dudatar / delilorn / tarivik / babadra: model widths to measure")
+                         "tarivik, babadra: beside Delilorn; gunulorn: beside Babadra")
+    ap.add_argument("--sizes", default="2048,4096", help="--arch dudatar / delilorn / tarivik / babadra / gunulorn: model widths to measure")
     a = ap.parse_args()
     if a.impl == "reference":
         return reference_main(a)

@@ -471,12 +471,27 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
           tmem_load32(tmem_o + lane_addr + c, v);
           if (p.turn.cos && valid && c < 2 * p.turn.half) {
             const size_t at = (size_t)pos * p.turn.half + (c >> 1);
+            if (p.turn.half % 16 == 0) {      // whole runs of 16 angles, 16 bytes at a time
 #pragma unroll
-            for (int e = 0; e < 32; e += 2) {
-              if (c + e < 2 * p.turn.half) {
-                const float cs = p.turn.cos[at + e / 2], sn = p.turn.sin[at + e / 2], a = v[e], b = v[e + 1];
-                v[e] = a * cs + b * sn;
-                v[e + 1] = b * cs - a * sn;
+              for (int e = 0; e < 32; e += 8) {
+                const float4 cs = *reinterpret_cast<const float4*>(p.turn.cos + at + e / 2);
+                const float4 sn = *reinterpret_cast<const float4*>(p.turn.sin + at + e / 2);
+                const float cv[4] = {cs.x, cs.y, cs.z, cs.w}, sv4[4] = {sn.x, sn.y, sn.z, sn.w};
+#pragma unroll
+                for (int k = 0; k < 4; ++k) {
+                  const float a = v[e + 2 * k], b = v[e + 2 * k + 1];
+                  v[e + 2 * k] = a * cv[k] + b * sv4[k];
+                  v[e + 2 * k + 1] = b * cv[k] - a * sv4[k];
+                }
+              }
+            } else {
+#pragma unroll
+              for (int e = 0; e < 32; e += 2) {
+                if (c + e < 2 * p.turn.half) {
+                  const float cs = p.turn.cos[at + e / 2], sn = p.turn.sin[at + e / 2], a = v[e], b = v[e + 1];
+                  v[e] = a * cs + b * sn;
+                  v[e + 1] = b * cs - a * sn;
+                }
               }
             }
           }
@@ -539,6 +554,7 @@ TS_EXPORT int ts_paged_attention_tcgen05(const void* q, void* out, const void* k
                                          int tile_queries, int keep_first, const float* sinks, int chunk,
                                          const float* slopes, float softcap, int v_share, const float* turn_cos,
                                          const float* turn_sin, int turn_half, const int* positions, cudaStream_t stream) {
+  TS_REQUIRE(turn_cos == nullptr || ((uintptr_t)turn_cos | (uintptr_t)turn_sin) % 16 == 0, "paged_attention_tcgen05: the angles must be 16-byte aligned");
   TS_REQUIRE(turn_cos == nullptr || (turn_sin && turn_half > 0 && 2 * turn_half <= D), "paged_attention_tcgen05: turned outputs of %d pairs in heads of %d", turn_half, D);
   TS_REQUIRE(keep_first >= 0, "paged_attention_tcgen05: keep_first %d", keep_first);
   TS_REQUIRE(v_share >= 1 && Hkv % v_share == 0, "paged_attention_tcgen05: %d key heads do not share values in runs of %d", Hkv, v_share);

@@ -146,19 +146,20 @@ __global__ void __launch_bounds__(CONV_THREADS) causal_conv_kernel(ConvParams p)
 // The rows x [T, H dim (q) | G dim (k) | G vdim (v)] of a fused projection pass the convolution and leave as what
 // the attention kernels read: query rows [T, H, stored] (times one factor per head), keys and values at the cache
 // slots of their tokens, heads padded with zeros to `stored`.  G = 0: queries only (the keys and values are
-// another layer's).  A thread owns VEC neighbouring columns of a stored head over CONV_TILE tokens of one request;
+// another layer's).  A thread owns VEC neighbouring columns of a stored head over HEADS_TILE tokens of one request,
+// whose loads are all in flight together (the tokens before them are read again: they come from L1 and L2);
 // the block of a request's first tile also replaces the request's state, as in causal_conv_kernel.
 struct ConvHeads {
   const void* x; long long ldx;
-  VecParam w;                       // [channels, TAPS]; null (TAPS 1): the rows as they are
+  VecParam w;                       // [TAPS, channels], so that a warp's loads are contiguous; null (TAPS 1): the rows as they are
   VecParam factor;                  // [H] or null
   float* state;                     // [slots, TAPS - 1, channels]
   const int* state_slots; const int* fresh; const int* cu_q;
-  int H, G, dim, vdim, stored, page_size, channels;
+  int H, G, dim, vdim, stored, page_size, page_shift, channels;     // page_shift: log2(page_size), or -1
   void* q_out; void* k_cache; void* v_cache;
   const int* slot_mapping;
 };
-constexpr int CONV_BATCH = 8;        // tokens whose loads are in flight together
+constexpr int HEADS_TILE = 8;        // tokens of a block: at least CONV_MAX_TAPS - 1
 
 template <typename T, int VEC> struct Pack;
 template <> struct Pack<float, 1> {
@@ -202,80 +203,91 @@ __global__ void __launch_bounds__(CONV_THREADS) conv_heads_kvwrite_kernel(ConvHe
   float factor = 1.f;
   if (real) {      // (weights are constants: fetched while the predecessor still runs)
 #pragma unroll
-    for (int j = 0; j < TAPS; ++j)
+    for (int j = 0; j < TAPS; ++j) {
+      const size_t at = (size_t)j * p.channels + c;
+      if (p.w.ptr == nullptr) {
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) w[j][e] = p.w.ptr ? p.w[(c + e) * TAPS + j] : 1.f;
+        for (int e = 0; e < VEC; ++e) w[j][e] = 1.f;
+      } else if (p.w.is_f32) {
+        Pack<float, VEC>::load(static_cast<const float*>(p.w.ptr) + at, w[j]);
+      } else {
+        Pack<__nv_bfloat16, VEC>::load(static_cast<const __nv_bfloat16*>(p.w.ptr) + at, w[j]);
+      }
+    }
     if (is_q && p.factor.ptr) factor = p.factor[head];
   }
   pdl_wait();
   const int b = blockIdx.z;
   const int t0 = p.cu_q[b], n = p.cu_q[b + 1] - t0;
-  const int first = blockIdx.y * CONV_TILE;
+  const int first = blockIdx.y * HEADS_TILE;
   if (first >= n || !live) return;
+  const int count = min(HEADS_TILE, n - first);
+  const int tok = t0 + first;
+  // where token k's result goes: the query row, or the token's place in the cache (null: nowhere)
+  T* const q_row = static_cast<T*>(p.q_out) + ((size_t)tok * p.H + head) * p.stored + d;
+  T* const cache = static_cast<T*>(is_v ? p.v_cache : p.k_cache) + d;
+  auto place = [&](int k) -> T* {
+    if (is_q) return q_row + (size_t)k * p.H * p.stored;
+    const int slot = p.slot_mapping[tok + k];
+    if (slot < 0) return nullptr;
+    const int page = p.page_shift >= 0 ? slot >> p.page_shift : slot / p.page_size;
+    return cache + ((size_t)(page * p.G + g) * p.page_size + (slot - page * p.page_size)) * p.stored;
+  };
+  if (!real) {
+    const float zeros[VEC] = {};
+    for (int k = 0; k < count; ++k)
+      if (T* dst = place(k)) Pack<T, VEC>::store(dst, zeros);
+    return;
+  }
   const T* x = static_cast<const T*>(p.x) + c;
+  const T* row = x + (size_t)tok * p.ldx;
+  // in[i] = input at token first - H1 + i of this portion (before the portion: the state)
+  float in[H1 + HEADS_TILE][VEC];
+  T* dst[HEADS_TILE];
+#pragma unroll
+  for (int k = 0; k < HEADS_TILE; ++k)
+    if (k < count) {
+      Pack<T, VEC>::load(row + (size_t)k * p.ldx, in[H1 + k]);
+      dst[k] = place(k);
+    }
   float* st = nullptr;
-  float hist[H1 > 0 ? H1 : 1][VEC];
   bool is_fresh = false;
-  if (H1 > 0 && real) {
-    st = p.state + (size_t)p.state_slots[b] * H1 * p.channels + c;
-    is_fresh = p.fresh[b] != 0;
+  if (H1 > 0) {
+    if (first == 0) {
+      st = p.state + (size_t)p.state_slots[b] * H1 * p.channels + c;
+      is_fresh = p.fresh[b] != 0;
 #pragma unroll
-    for (int i = 0; i < H1; ++i) {       // hist[i] = input at token first - H1 + i of this portion (before it: the state)
-      if (first == 0) {
+      for (int i = 0; i < H1; ++i)
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) hist[i][e] = is_fresh ? 0.f : st[(size_t)i * p.channels + e];
-      } else {
-        Pack<T, VEC>::load(x + (size_t)(t0 + first - H1 + i) * p.ldx, hist[i]);
-      }
+        for (int e = 0; e < VEC; ++e) in[i][e] = is_fresh ? 0.f : st[(size_t)i * p.channels + e];
+    } else {
+#pragma unroll
+      for (int i = 0; i < H1; ++i) Pack<T, VEC>::load(row - (size_t)(H1 - i) * p.ldx, in[i]);
     }
   }
-  const int last = min(n, first + CONV_TILE);
-  for (int tok0 = first; tok0 < last; tok0 += CONV_BATCH) {
-    float in[CONV_BATCH][VEC];
-    int slot[CONV_BATCH];
 #pragma unroll
-    for (int k = 0; k < CONV_BATCH; ++k) {
-      if (tok0 + k < last) {
-        if (real) Pack<T, VEC>::load(x + (size_t)(t0 + tok0 + k) * p.ldx, in[k]);
-        slot[k] = is_q ? 0 : p.slot_mapping[t0 + tok0 + k];
-      }
-    }
-#pragma unroll
-    for (int k = 0; k < CONV_BATCH; ++k) {
-      if (tok0 + k >= last) break;
+  for (int k = 0; k < HEADS_TILE; ++k) {
+    if (k < count && dst[k] != nullptr) {
       float y[VEC];
 #pragma unroll
       for (int e = 0; e < VEC; ++e) {
-        float acc = 0.f;
-        if (real) {
-          acc = w[H1][e] * in[k][e];
+        float acc = w[H1][e] * in[H1 + k][e];
 #pragma unroll
-          for (int i = 0; i < H1; ++i) acc = fmaf(w[i][e], hist[i][e], acc);
-          acc *= factor;
-#pragma unroll
-          for (int i = 0; i + 1 < H1; ++i) hist[i][e] = hist[i + 1][e];
-          if (H1 > 0) hist[H1 - 1][e] = in[k][e];
-        }
-        y[e] = acc;
+        for (int i = 0; i < H1; ++i) acc = fmaf(w[i][e], in[k + i][e], acc);
+        y[e] = acc * factor;
       }
-      if (is_q) {
-        Pack<T, VEC>::store(static_cast<T*>(p.q_out) + ((size_t)(t0 + tok0 + k) * p.H + head) * p.stored + d, y);
-      } else if (slot[k] >= 0) {
-        const size_t page = slot[k] / p.page_size, in_page = slot[k] % p.page_size;
-        T* cache = static_cast<T*>(is_v ? p.v_cache : p.k_cache);
-        Pack<T, VEC>::store(cache + ((page * p.G + g) * p.page_size + in_page) * p.stored + d, y);
-      }
+      Pack<T, VEC>::store(dst[k], y);
     }
   }
-  if (H1 > 0 && first == 0 && real) {
+  if (H1 > 0 && first == 0) {
     // new state: inputs at tokens n - H1 .. n - 1; tokens below 0 are the old state's row i + n, which an ascending
     // walk has not overwritten yet
 #pragma unroll
     for (int i = 0; i < H1; ++i) {
-      const int tok = n - H1 + i;
+      const int at = n - H1 + i;
       float v[VEC];
-      if (tok >= 0) {
-        Pack<T, VEC>::load(x + (size_t)(t0 + tok) * p.ldx, v);
+      if (at >= 0) {
+        Pack<T, VEC>::load(x + (size_t)(t0 + at) * p.ldx, v);
       } else {
 #pragma unroll
         for (int e = 0; e < VEC; ++e) v[e] = is_fresh ? 0.f : st[(size_t)(i + n) * p.channels + e];
@@ -613,7 +625,7 @@ TS_EXPORT int ts_causal_conv(const void* x, long long ldx, int x_is_f32, void* y
   return 0;
 }
 
-// x [T, H dim | G dim | G vdim]; w [channels, taps] or null (taps 1); factor [H] or null; G 0: queries only
+// x [T, H dim | G dim | G vdim]; w [taps, channels] or null (taps 1); factor [H] or null; G 0: queries only
 TS_EXPORT int ts_conv_heads_kvwrite(int is_f32, const void* x, long long ldx, const void* w, int w_is_f32, int taps,
                                     const void* factor, int factor_is_f32, float* state, const int* state_slots,
                                     const int* fresh, const int* cu_q, int num_requests, int max_q_len, int H, int G, int dim,
@@ -625,10 +637,12 @@ TS_EXPORT int ts_conv_heads_kvwrite(int is_f32, const void* x, long long ldx, co
   TS_REQUIRE(x && q_out && (taps == 1 || state) && state_slots && fresh && cu_q, "conv_heads_kvwrite: a null operand");
   TS_REQUIRE(G == 0 || (k_cache && v_cache && slot_mapping && page_size > 0), "conv_heads_kvwrite: no cache to write");
   ConvHeads p{x, ldx, VecParam{w, w_is_f32}, VecParam{factor, factor_is_f32}, state, state_slots, fresh, cu_q, H, G, dim, vdim, stored,
-              page_size, H * dim + G * (dim + vdim), q_out, k_cache, v_cache, slot_mapping};
-  const bool even = dim % 2 == 0 && vdim % 2 == 0 && stored % 2 == 0 && ldx % 2 == 0 && (uintptr_t)x % 8 == 0;
+              page_size, -1, H * dim + G * (dim + vdim), q_out, k_cache, v_cache, slot_mapping};
+  if (page_size > 0 && (page_size & (page_size - 1)) == 0)
+    for (p.page_shift = 0; (1 << p.page_shift) < page_size;) ++p.page_shift;
+  const bool even = dim % 2 == 0 && vdim % 2 == 0 && stored % 2 == 0 && ldx % 2 == 0 && ((uintptr_t)x | (uintptr_t)w) % 8 == 0;
   const int cols = (H + 2 * G) * stored / (even ? 2 : 1);
-  const dim3 grid((cols + CONV_THREADS - 1) / CONV_THREADS, (max_q_len + CONV_TILE - 1) / CONV_TILE, num_requests);
+  const dim3 grid((cols + CONV_THREADS - 1) / CONV_THREADS, (max_q_len + HEADS_TILE - 1) / HEADS_TILE, num_requests);
   TS_REQUIRE(grid.y <= 65535 && grid.z <= 65535, "conv_heads_kvwrite: the step is too large");
   if (is_f32) return even ? launch_conv_heads<float, 2>(p, taps, grid, stream) : launch_conv_heads<float, 1>(p, taps, grid, stream);
   return even ? launch_conv_heads<__nv_bfloat16, 2>(p, taps, grid, stream) : launch_conv_heads<__nv_bfloat16, 1>(p, taps, grid, stream);

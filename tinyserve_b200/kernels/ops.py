@@ -2225,15 +2225,15 @@ def poly_norm(z, coefficients, eps):
 def conv_heads_kvwrite(x, ctx, num_heads, num_kv_heads, dim, vdim, stored_dim, weight=None, state=None, factor=None,
                        k_cache=None, v_cache=None, slot_mapping=None, page_size=0):
     """The rows x [T, H dim | G dim | G vdim] of a fused q/k/v projection through a causal convolution over
-    time on every channel (``weight`` [channels, taps], ``state`` float32 [slots, taps - 1, channels] as for
-    ``causal_conv``; None: as they are): returns the query rows [T, H, stored_dim], head h times factor[h]
+    time on every channel (``weight`` [taps, channels], oldest tap first; ``state`` float32 [slots, taps - 1,
+    channels] as for ``causal_conv``; None: as they are): returns the query rows [T, H, stored_dim], head h times factor[h]
     (``factor`` [H] or None), and writes keys and values to the cache slots of ``slot_mapping``, heads
     padded with zeros.  Without ``slot_mapping`` x holds the queries' columns only."""
     G = num_kv_heads if slot_mapping is not None else 0
     channels = num_heads * dim + G * (dim + vdim)
-    taps = weight.shape[1] if weight is not None else 1
+    taps = weight.shape[0] if weight is not None else 1
     _cuda(x, weight, state, factor, k_cache, v_cache, slot_mapping)
-    if x.shape[1] != channels or x.stride(1) != 1 or (weight is not None and (weight.shape[0] != channels or not weight.is_contiguous())):
+    if x.shape[1] != channels or x.stride(1) != 1 or (weight is not None and (weight.shape[1] != channels or not weight.is_contiguous())):
         raise ValueError("conv_heads_kvwrite: the projection and the convolution do not have heads x size channels")
     if not 1 <= taps <= CAUSAL_CONV_MAX_TAPS:
         raise ValueError(f"conv_heads_kvwrite: 1 to {CAUSAL_CONV_MAX_TAPS} taps, got {taps}")

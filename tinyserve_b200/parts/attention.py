@@ -192,6 +192,8 @@ class Attention(Mixer):
         tensors = dict(tensors)
         if self.bias and self.gate_size and "qkv_proj.bias" in tensors:
             tensors["qkv_proj.bias"][self.q_size + self.kv_size + self.v_size:] = 0
+        if "qkv_conv.weight" in tensors:
+            tensors["qkv_conv.weight"] = tensors["qkv_conv.weight"].t().contiguous()       # tap by tap: [taps, channels]
         if "sinks" in tensors:
             tensors["sinks"] = tensors["sinks"].float().contiguous()       # they join a 32-bit sum
         if self.differential and "lambda_q1" in tensors:
