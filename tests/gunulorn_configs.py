@@ -51,7 +51,7 @@ GUNULORN_TINY = {
         "layers": [
             {"type": "attention", "mlp": _dense(192), "mixer": _conv(8, 2, 64, 64, 0.125, 2)},
             {"type": "attention", "mlp": _moe(64, 8, 2, 3), "mixer": _conv(8, 2, 64, 64, 0.2, 6, kv_from=0)},
-            {"type": "attention_2", "mlp": _moe(32, 12, 4, 5), "mixer": _turned(8, 2, 64, 64, 0.125, 1e4, 32, 40, 2)},
+            {"type": "attention_2", "mlp": _moe(32, 10, 3, 5), "mixer": _turned(6, 3, 64, 64, 0.15, 1e4, 48, 40, 2)},
             {"type": "attention_2", "mlp": _dense(96), "mixer": _turned(2, 1, 32, 64, 0.2, 2.5e5, 16, 64, 17)},
             {"type": "attention", "mlp": _moe(64, 4, 4, 2), "mixer": _conv(8, 2, 64, 64, 0.125, 3, kv_from=0)},
         ]},

@@ -753,7 +753,7 @@ __device__ __forceinline__ void attn_decode_body(const MmaAttnParams& p, const C
     return p.turn.value(v, mate, d, qpos);
   };
   for (int i = threadIdx.x; i < ng * D; i += THREADS) {
-    const unsigned lanes = ~0u >> (32 - min(32, ng * D - (i - lane)));        // the warp's lanes of this round
+    const unsigned lanes = ~0u >> (32 - min(32, ng * D - (i - lane)));        // the warp's lanes that take part
     const int r = i / D, d = i % D;
     float mx = -INFINITY;
 #pragma unroll

@@ -698,9 +698,21 @@ __device__ __forceinline__ void poly_sums(float z, float& s2, float& s4, float& 
   s6 = fmaf(q2, q, s6);
 }
 
+// sums of three values over the block in one exchange; `scratch` holds 96 floats
+__device__ __forceinline__ void block_sum3(float& a, float& b, float& c, float* scratch) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = (blockDim.x + 31) >> 5;
+  a = warp_sum(a); b = warp_sum(b); c = warp_sum(c);
+  if (lane == 0) { scratch[warp] = a; scratch[32 + warp] = b; scratch[64 + warp] = c; }
+  __syncthreads();
+  // (every warp adds the warps' sums itself: the same order, the same result)
+  a = warp_sum(lane < warps ? scratch[lane] : 0.f);
+  b = warp_sum(lane < warps ? scratch[32 + lane] : 0.f);
+  c = warp_sum(lane < warps ? scratch[64 + lane] : 0.f);
+}
+
 template <typename T, int HOLD>      // HOLD 0: any row length and alignment, element by element
 __global__ void poly_norm_kernel(const T* __restrict__ z, T* __restrict__ out, VecParam coef, float eps, int n) {
-  __shared__ float scratch[33];
+  __shared__ float scratch[96];
   pdl_trigger();
   pdl_wait();
   const T* row = z + (size_t)blockIdx.x * n;
@@ -708,7 +720,7 @@ __global__ void poly_norm_kernel(const T* __restrict__ z, T* __restrict__ out, V
   float s2 = 0.f, s4 = 0.f, s6 = 0.f;
   if constexpr (HOLD == 0) {
     for (int c = threadIdx.x; c < n; c += blockDim.x) poly_sums(to_f32<T>(row[c]), s2, s4, s6);
-    s2 = block_sum(s2, scratch); s4 = block_sum(s4, scratch); s6 = block_sum(s6, scratch);
+    block_sum3(s2, s4, s6, scratch);
     const PolyFactors f = poly_factors(s2, s4, s6, coef, n, eps);
     for (int c = threadIdx.x; c < n; c += blockDim.x) dst[c] = from_f32<T>(poly_value(to_f32<T>(row[c]), f));
   } else {
@@ -735,7 +747,7 @@ __global__ void poly_norm_kernel(const T* __restrict__ z, T* __restrict__ out, V
 #pragma unroll
       for (int e = 0; e < N; ++e) poly_sums(v[e], s2, s4, s6);
     }
-    s2 = block_sum(s2, scratch); s4 = block_sum(s4, scratch); s6 = block_sum(s6, scratch);
+    block_sum3(s2, s4, s6, scratch);
     const PolyFactors f = poly_factors(s2, s4, s6, coef, n, eps);
     auto put = [&](int c, const uint4& raw) {
       float v[N];
