@@ -100,6 +100,9 @@ class ModelSpec:
     logit_softcap: float = 0.0
     # the embedding rows are multiplied by this on their way into the 32-bit stream
     embedding_scale: float = 1.0
+    # parallel residual streams, all equal to the embedding output at the start, whose sum goes to the final norm
+    # (the layers' arrangement must keep them: "hyper_connections"); 0: one residual
+    streams: int = 0
     # operations on the residual stream between blocks, by name: ((name, PartSpec), ...); a
     # ``LayerCall.before`` says where one runs.  Its tensors live under "{prefix}{name}"
     stream_ops: tuple = ()

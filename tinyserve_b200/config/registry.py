@@ -16,6 +16,7 @@ from .delilorn import DelilornConfig
 from .dudatar import DudatarConfig
 from .gunulorn import GunulornConfig
 from .model_config import ConfigError, ModelConfig, Qwen3Config
+from .ronolorn import RonolornConfig
 from .tarivik import TarivikConfig
 
 ARCHITECTURES: dict[str, type] = {}
@@ -68,3 +69,4 @@ register_architecture(DelilornConfig.architecture, DelilornConfig)
 register_architecture(TarivikConfig.architecture, TarivikConfig)
 register_architecture(BabadraConfig.architecture, BabadraConfig)
 register_architecture(GunulornConfig.architecture, GunulornConfig)
+register_architecture(RonolornConfig.architecture, RonolornConfig)

@@ -231,6 +231,52 @@ __device__ __forceinline__ float gated_value(float g, float u, int act, float li
   return activate(g, act) * u;
 }
 
+// feed-forward without a gate: act(x)
+enum { PLAIN_NONE = 0, PLAIN_RELU_SQUARED = 1, PLAIN_COUNT = 2 };
+__device__ __forceinline__ float plain_value(float x, int act) {
+  if (act == PLAIN_RELU_SQUARED) {
+    x = fmaxf(x, 0.f);
+    return x * x;
+  }
+  return x;
+}
+
+// eight neighbouring elements, 16-byte aligned
+template <typename T> __device__ __forceinline__ void load8(const T* p, float (&v)[8]);
+template <> __device__ __forceinline__ void load8<float>(const float* p, float (&v)[8]) {
+  const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+template <> __device__ __forceinline__ void load8<__nv_bfloat16>(const __nv_bfloat16* p, float (&v)[8]) {
+  const uint4 raw = *reinterpret_cast<const uint4*>(p);
+  const __nv_bfloat162* e = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) { v[2 * i] = __low2float(e[i]); v[2 * i + 1] = __high2float(e[i]); }
+}
+template <typename T> __device__ __forceinline__ void store8(T* p, const float (&v)[8]);
+template <> __device__ __forceinline__ void store8<float>(float* p, const float (&v)[8]) {
+  reinterpret_cast<float4*>(p)[0] = make_float4(v[0], v[1], v[2], v[3]);
+  reinterpret_cast<float4*>(p)[1] = make_float4(v[4], v[5], v[6], v[7]);
+}
+template <> __device__ __forceinline__ void store8<__nv_bfloat16>(__nv_bfloat16* p, const float (&v)[8]) {
+  uint4 raw;
+  __nv_bfloat162* e = reinterpret_cast<__nv_bfloat162*>(&raw);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) e[i] = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+  *reinterpret_cast<uint4*>(p) = raw;
+}
+// the four neighbouring pairs of eight elements turned by the angles whose cos / sin lie at `at`
+__device__ __forceinline__ void turn_pairs8(float (&v)[8], const float* __restrict__ cos, const float* __restrict__ sin, size_t at) {
+  const float4 c = *reinterpret_cast<const float4*>(cos + at), s = *reinterpret_cast<const float4*>(sin + at);
+  const float cs[4] = {c.x, c.y, c.z, c.w}, sn[4] = {s.x, s.y, s.z, s.w};
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const float a = v[2 * i], b = v[2 * i + 1];
+    v[2 * i] = a * cs[i] - b * sn[i];
+    v[2 * i + 1] = b * cs[i] + a * sn[i];
+  }
+}
+
 // a weight vector that is either float or bfloat16, chosen at run time
 struct VecParam {
   const void* ptr;

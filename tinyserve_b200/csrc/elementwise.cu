@@ -951,6 +951,55 @@ TS_EXPORT int ts_gated_activation(int dtype, const void* in, void* out, int num_
   return ts_fail("gated_activation: unknown dtype %d", dtype);
 }
 
+// ------------------------------------------------------------------ activation without a gate, in place
+template <typename T>
+__global__ void plain_activation_kernel(T* __restrict__ x, long long count, int act) {
+  pdl_trigger();
+  pdl_wait();
+  const long long step = (long long)gridDim.x * blockDim.x;
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < count; i += step) x[i] = from_f32<T>(plain_value(to_f32<T>(x[i]), act));
+}
+// a thread has PLAIN_PACKS runs of eight elements in flight
+constexpr int PLAIN_PACKS = 4;
+template <typename T>
+__global__ void __launch_bounds__(256) plain_activation_vec_kernel(T* __restrict__ x, long long packs, int act) {
+  pdl_trigger();
+  pdl_wait();
+  const long long first = blockIdx.x * (long long)(256 * PLAIN_PACKS) + threadIdx.x;
+  float v[PLAIN_PACKS][8];
+#pragma unroll
+  for (int j = 0; j < PLAIN_PACKS; ++j)
+    if (first + 256 * j < packs) load8<T>(x + (first + 256 * j) * 8, v[j]);
+#pragma unroll
+  for (int j = 0; j < PLAIN_PACKS; ++j) {
+    if (first + 256 * j >= packs) continue;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) v[j][e] = plain_value(v[j][e], act);
+    store8<T>(x + (first + 256 * j) * 8, v[j]);
+  }
+}
+
+template <typename T>
+int launch_plain_activation(void* x, long long count, int act, cudaStream_t stream) {
+  if (count % 8 == 0 && (uintptr_t)x % 16 == 0) {
+    const long long packs = count / 8, per = 256 * PLAIN_PACKS;
+    TS_LAUNCH("plain_activation", plain_activation_vec_kernel<T>, (unsigned)((packs + per - 1) / per), 256, 0, stream, (T*)x, packs, act);
+  } else {
+    const long long blocks = (count + 255) / 256;
+    TS_LAUNCH("plain_activation", plain_activation_kernel<T>, (unsigned)(blocks < 148 * 16 ? blocks : 148 * 16), 256, 0, stream, (T*)x, count, act);
+  }
+  return 0;
+}
+
+// x [count] <- act(x)
+TS_EXPORT int ts_plain_activation(int dtype, void* x, long long count, int act, cudaStream_t stream) {
+  TS_REQUIRE(count > 0 && x, "plain_activation: empty input");
+  TS_REQUIRE(act > 0 && act < PLAIN_COUNT, "plain_activation: unknown activation %d", act);
+  if (dtype == TS_F32) return launch_plain_activation<float>(x, count, act, stream);
+  if (dtype == TS_BF16) return launch_plain_activation<__nv_bfloat16>(x, count, act, stream);
+  return ts_fail("plain_activation: unknown dtype %d", dtype);
+}
+
 // ------------------------------------------------------------------ q/k norm + rotary + cache write
 // qkv [T, (H + 2 Hkv) * D]: q heads, k heads, v heads.  One warp per (token, head):
 //   q heads: optional RMSNorm over D, rotary, stored to q_out [T, H, D];
@@ -1821,43 +1870,6 @@ __global__ void rope_unit_kvwrite_kernel(const T* __restrict__ q, long long ldq,
 
 // The same for neighbouring pairs without norms and maps, sizes in multiples of 8: a thread turns eight columns of a
 // stored head (four pairs), 16 bytes of bfloat16 or two times 16 bytes of float in and out.
-template <typename T>
-__device__ __forceinline__ void load8(const T* p, float (&v)[8]);
-template <>
-__device__ __forceinline__ void load8<float>(const float* p, float (&v)[8]) {
-  const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
-  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
-}
-template <>
-__device__ __forceinline__ void load8<__nv_bfloat16>(const __nv_bfloat16* p, float (&v)[8]) {
-  chunk16_floats<__nv_bfloat16>(*reinterpret_cast<const uint4*>(p), v);
-}
-template <typename T>
-__device__ __forceinline__ void store8(T* p, const float (&v)[8]);
-template <>
-__device__ __forceinline__ void store8<float>(float* p, const float (&v)[8]) {
-  reinterpret_cast<float4*>(p)[0] = make_float4(v[0], v[1], v[2], v[3]);
-  reinterpret_cast<float4*>(p)[1] = make_float4(v[4], v[5], v[6], v[7]);
-}
-template <>
-__device__ __forceinline__ void store8<__nv_bfloat16>(__nv_bfloat16* p, const float (&v)[8]) {
-  uint4 raw;
-  __nv_bfloat162* e = reinterpret_cast<__nv_bfloat162*>(&raw);
-#pragma unroll
-  for (int i = 0; i < 4; ++i) e[i] = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
-  *reinterpret_cast<uint4*>(p) = raw;
-}
-__device__ __forceinline__ void turn_pairs8(float (&v)[8], const float* __restrict__ cos, const float* __restrict__ sin, size_t at) {
-  const float4 c = *reinterpret_cast<const float4*>(cos + at), s = *reinterpret_cast<const float4*>(sin + at);
-  const float cs[4] = {c.x, c.y, c.z, c.w}, sn[4] = {s.x, s.y, s.z, s.w};
-#pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    const float a = v[2 * i], b = v[2 * i + 1];
-    v[2 * i] = a * cs[i] - b * sn[i];
-    v[2 * i + 1] = b * cs[i] + a * sn[i];
-  }
-}
-
 template <typename T>
 __global__ void rope_pairs_kvwrite_kernel(const T* __restrict__ q, long long ldq, const T* __restrict__ k, long long ldk,
                                           const T* __restrict__ v, long long ldv, T* __restrict__ q_out,

@@ -77,6 +77,7 @@ struct GemmParams {
   int gated_act;        // 0: off; else the activation's code + 1
   float gated_limit;    // the bound of a bounded activation (gated_value)
   VecParam bias;        // [N] added to every token's result (plain output only); ptr null: none
+  int out_act;          // plain output of one product: the activation (PLAIN_*) the result passes, after the bias
   VecParam res_scale;   // residual form: [N] factors on the result before it joins the residual; ptr null: none
   // the forms with several operand pairs (Maps3)
   int segments;         // beside: how many products; 0: chained
@@ -367,7 +368,7 @@ gemm_wx_kernel(const __grid_constant__ MAPS maps, const __grid_constant__ GemmPa
         for (int i = 0; i < 8; ++i) v[i] *= row_scale[c + i];
       }
 #pragma unroll
-      for (int i = 0; i < 8; ++i) v[i] += bn;
+      for (int i = 0; i < 8; ++i) v[i] = plain_value(v[i] + bn, p.out_act);
       if (epi && n < N) {
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
@@ -428,8 +429,9 @@ gemm_wx_kernel(const __grid_constant__ MAPS maps, const __grid_constant__ GemmPa
             for (int i = 0; i < 8; ++i) {
               const int m = t0 + c0 + i;
               if (m < p.M) {
-                if (out_f32) static_cast<float*>(out)[(size_t)m * ldc + n] = sum[i];
-                else static_cast<bf16*>(out)[(size_t)m * ldc + n] = __float2bfloat16_rn(sum[i]);
+                const float y = plain_value(sum[i], p.out_act);
+                if (out_f32) static_cast<float*>(out)[(size_t)m * ldc + n] = y;
+                else static_cast<bf16*>(out)[(size_t)m * ldc + n] = __float2bfloat16_rn(y);
               }
             }
           }
@@ -515,17 +517,18 @@ int gemm_tiled(const void* x, const void* w, void* out, int M, int N, int K, lon
                long long ldc, int out_f32, int splits, float* partials, int* counters, const float* x_sumsq,
                int x_tiles, float x_eps, float* residual, const void* norm_w, int norm_w_is_f32, void* hprime,
                float* sumsq_out, int gated_act, const void* bias, int bias_is_f32, float gated_limit,
-               const void* res_scale, int res_scale_is_f32, cudaStream_t stream);
+               const void* res_scale, int res_scale_is_f32, int out_act, cudaStream_t stream);
 }
 
 // bias: [N] float or bfloat16 (bias_is_f32), added to every token's result; needs an output
-// (not with out == nullptr, where only partial tiles are produced).  nullptr: none.
+// (not with out == nullptr, where only partial tiles are produced).  nullptr: none.  act: PLAIN_* on the result.
 TS_EXPORT int ts_gemm_tcgen05(const void* x, const void* w, void* out, int M, int N, int K, long long ldx,
                               long long ldw, long long ldc, int out_f32, int splits, float* partials,
-                              int* counters, const void* bias, int bias_is_f32, cudaStream_t stream) {
-  TS_REQUIRE(bias == nullptr || out != nullptr, "gemm_tcgen05: a bias needs an output, not partial tiles only");
+                              int* counters, const void* bias, int bias_is_f32, int act, cudaStream_t stream) {
+  TS_REQUIRE((bias == nullptr && act == PLAIN_NONE) || out != nullptr, "gemm_tcgen05: a bias or an activation needs an output, not partial tiles only");
+  TS_REQUIRE(act >= 0 && act < PLAIN_COUNT, "gemm_tcgen05: unknown activation %d", act);
   return gemm_tiled(x, w, out, M, N, K, ldx, ldw, ldc, out_f32, splits, partials, counters, nullptr, 0, 0.f,
-                    nullptr, nullptr, 0, nullptr, nullptr, 0, bias, bias_is_f32, 0.f, nullptr, 0, stream);
+                    nullptr, nullptr, 0, nullptr, nullptr, 0, bias, bias_is_f32, 0.f, nullptr, 0, act, stream);
 }
 
 // The same product with extras.  The first two are for up to 16 tokens.
@@ -556,7 +559,7 @@ TS_EXPORT int ts_gemm_tcgen05_fused(const void* x, const void* w, void* out, int
              "gemm_tcgen05: the residual form needs the norm's weight, both outputs and at most 8 cuts");
   return gemm_tiled(x, w, out, M, N, K, ldx, ldw, ldc, out_f32, splits, partials, counters, x_sumsq, x_tiles,
                     x_eps, residual, norm_w, norm_w_is_f32, hprime, sumsq_out, gated_act, nullptr, 0, gated_limit,
-                    residual ? res_scale : nullptr, res_scale_is_f32, stream);
+                    residual ? res_scale : nullptr, res_scale_is_f32, PLAIN_NONE, stream);
 }
 
 namespace {
@@ -564,7 +567,7 @@ int gemm_tiled(const void* x, const void* w, void* out, int M, int N, int K, lon
                long long ldc, int out_f32, int splits, float* partials, int* counters, const float* x_sumsq,
                int x_tiles, float x_eps, float* residual, const void* norm_w, int norm_w_is_f32, void* hprime,
                float* sumsq_out, int gated_act, const void* bias, int bias_is_f32, float gated_limit,
-               const void* res_scale, int res_scale_is_f32, cudaStream_t stream) {
+               const void* res_scale, int res_scale_is_f32, int out_act, cudaStream_t stream) {
   TS_REQUIRE(M > 0 && N > 0 && K > 0, "gemm_tcgen05: empty operand");
   TS_REQUIRE(M <= 65535 * 128, "gemm_tcgen05: too many rows");
   TS_REQUIRE(K % 8 == 0 && ldx % 8 == 0 && ldw % 8 == 0, "gemm_tcgen05: K and the leading dimensions must be multiples of 8 (16-byte rows for TMA), got K=%d", K);
@@ -584,6 +587,7 @@ int gemm_tiled(const void* x, const void* w, void* out, int M, int N, int K, lon
   p.hprime = static_cast<bf16*>(hprime); p.sumsq_out = sumsq_out;
   p.gated_act = gated_act;
   p.gated_limit = gated_limit;
+  p.out_act = out_act;
   p.bias = VecParam{bias, bias_is_f32};
   p.res_scale = VecParam{res_scale, res_scale_is_f32};
   dim3 grid((N + TILE_N - 1) / TILE_N, (M + tile_t - 1) / tile_t, splits);

@@ -16,7 +16,8 @@
 //  * ts_gate_columns: out[t, h * vdim + c] = x[t, h, c] * sigmoid(gate[t, h * vdim + c]) for heads
 //    stored wider than their values.
 //  * ts_joint_norm_kvwrite: q and k of a token normed over all their heads at once (one weight
-//    per column), q to padded rows for the attention kernels, k and v to the token's cache slot.
+//    per column), optionally rotated, q to padded rows for the attention kernels, k and v to the token's cache
+//    slot; v may be the k rows as they come.
 //  * ts_mlstm_gates: the stabilised gates of a matrix memory with exponential input gate:
 //    m_t = max(f_t + m_(t-1), i_t), keep_t = exp(f_t + m_(t-1) - m_t), write_t = exp(i_t - m_t),
 //    floor_t = exp(-m_t); i and f capped by cap tanh(. / cap), f through log-sigmoid; m is state.
@@ -382,6 +383,9 @@ struct JointNorm {
   void* k_cache; void* v_cache;     // [pages, G, page, stored]
   const int* slot_mapping;          // null: nothing is written
   int out_is_f32;
+  // rotary positions after the norm, on the first `rot` columns of every head (0: none); pairs (2i, 2i + 1), or (i, i + rot / 2)
+  const float* cos; const float* sin; const int* positions;
+  int rot, interleaved;
 };
 
 __global__ void joint_norm_kvwrite_kernel(JointNorm p) {
@@ -389,7 +393,7 @@ __global__ void joint_norm_kvwrite_kernel(JointNorm p) {
   pdl_trigger();
   pdl_wait();
   const size_t t = blockIdx.x;
-  const int nq = p.H * p.dim, nk = p.G * p.dim;
+  const int nq = p.H * p.dim, nk = p.G * p.dim, half = p.rot >> 1;
   float aq = 0.f, ak = 0.f;
   if (p.qw.ptr) {
     for (int i = threadIdx.x; i < nq; i += blockDim.x) { const float v = p.q.at(t, i); aq = fmaf(v, v, aq); }
@@ -397,15 +401,25 @@ __global__ void joint_norm_kvwrite_kernel(JointNorm p) {
   }
   const float rq = p.qw.ptr ? rsqrtf(block_sum(aq, scratch) / (float)nq + p.eps) : 1.f;
   const float rk = p.qw.ptr ? rsqrtf(block_sum(ak, scratch) / (float)nk + p.eps) : 1.f;
+  const size_t angles = p.rot > 0 ? (size_t)p.positions[t] * half : 0;
+  // column d of the head at `base` of x's row, normed and rotated
+  auto element = [&](const Rows& x, const VecParam& w, float r, int base, int d) {
+    auto normed = [&](int e) {
+      const float v = x.at(t, base + e) * r;
+      return w.ptr ? v * w[base + e] : v;
+    };
+    const float a = normed(d);
+    if (d >= p.rot) return a;
+    const int j = p.interleaved ? d >> 1 : (d < half ? d : d - half);
+    const bool first = p.interleaved ? !(d & 1) : d < half;
+    const float b = normed(p.interleaved ? d ^ 1 : (first ? d + half : d - half));
+    const float c = p.cos[angles + j], s = p.sin[angles + j];
+    return first ? a * c - b * s : a * c + b * s;
+  };
   RowsOut qo{p.q_out, (long long)p.H * p.stored, p.out_is_f32};
   for (int i = threadIdx.x; i < p.H * p.stored; i += blockDim.x) {
     const int h = i / p.stored, d = i % p.stored;
-    float v = 0.f;
-    if (d < p.dim) {
-      v = p.q.at(t, h * p.dim + d) * rq;
-      if (p.qw.ptr) v *= p.qw[h * p.dim + d];
-    }
-    qo.put(t, i, v);
+    qo.put(t, i, d < p.dim ? element(p.q, p.qw, rq, h * p.dim, d) : 0.f);
   }
   if (!p.slot_mapping) return;
   const int slot = p.slot_mapping[t];
@@ -413,12 +427,8 @@ __global__ void joint_norm_kvwrite_kernel(JointNorm p) {
   const size_t page = slot / p.page_size, in_page = slot % p.page_size;
   for (int i = threadIdx.x; i < p.G * p.stored; i += blockDim.x) {
     const int g = i / p.stored, d = i % p.stored;
-    float kv = 0.f, vv = 0.f;
-    if (d < p.dim) {
-      kv = p.k.at(t, g * p.dim + d) * rk;
-      if (p.kw.ptr) kv *= p.kw[g * p.dim + d];
-    }
-    if (d < p.vdim) vv = p.v.at(t, g * p.vdim + d);
+    const float kv = d < p.dim ? element(p.k, p.kw, rk, g * p.dim, d) : 0.f;
+    const float vv = d < p.vdim ? p.v.at(t, g * p.vdim + d) : 0.f;
     const size_t at = ((page * p.G + g) * p.page_size + in_page) * p.stored + d;
     if (p.out_is_f32) {
       static_cast<float*>(p.k_cache)[at] = kv;
@@ -427,6 +437,88 @@ __global__ void joint_norm_kvwrite_kernel(JointNorm p) {
       static_cast<__nv_bfloat16*>(p.k_cache)[at] = __float2bfloat16_rn(kv);
       static_cast<__nv_bfloat16*>(p.v_cache)[at] = __float2bfloat16_rn(vv);
     }
+  }
+}
+
+// The same for sizes in multiples of 8 and neighbouring pairs: a thread keeps up to JOINT_PACKS runs of eight
+// columns of q and k between the sums and the results, 16 bytes of bfloat16 each.
+constexpr int JOINT_PACKS = 4, JOINT_THREADS = 256;
+
+__device__ __forceinline__ void weight8(const VecParam& w, int c, float (&v)[8]) {
+  if (w.is_f32) load8<float>(static_cast<const float*>(w.ptr) + c, v);
+  else load8<__nv_bfloat16>(static_cast<const __nv_bfloat16*>(w.ptr) + c, v);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(JOINT_THREADS) joint_norm_kvwrite_vec_kernel(JointNorm p) {
+  __shared__ float2 parts[JOINT_THREADS / 32];
+  pdl_trigger();
+  const int per = p.dim >> 3, packs_q = p.H * per, packs = packs_q + p.G * per;
+  pdl_wait();
+  const size_t t = blockIdx.x;
+  const T* q = static_cast<const T*>(p.q.ptr) + t * p.q.ld;
+  const T* k = static_cast<const T*>(p.k.ptr) + t * p.k.ld;
+  const T* v = static_cast<const T*>(p.v.ptr) + t * p.v.ld;
+  const int slot = p.slot_mapping ? p.slot_mapping[t] : -1;
+  const size_t angles = p.rot > 0 ? (size_t)p.positions[t] * (p.rot >> 1) : 0;
+  float x[JOINT_PACKS][8], aq = 0.f, ak = 0.f;
+#pragma unroll
+  for (int j = 0; j < JOINT_PACKS; ++j) {
+    const int i = threadIdx.x + j * blockDim.x;
+    if (i >= packs) continue;
+    const bool is_q = i < packs_q;
+    load8<T>(is_q ? q + i * 8 : k + (i - packs_q) * 8, x[j]);
+    float sum = 0.f;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) sum = fmaf(x[j][e], x[j][e], sum);
+    if (is_q) aq += sum;
+    else ak += sum;
+  }
+  aq = warp_sum(aq);
+  ak = warp_sum(ak);
+  if ((threadIdx.x & 31) == 0) parts[threadIdx.x >> 5] = make_float2(aq, ak);
+  __syncthreads();
+  aq = ak = 0.f;
+  for (int w = 0; w < (int)(blockDim.x >> 5); ++w) {
+    aq += parts[w].x;
+    ak += parts[w].y;
+  }
+  const float rq = rsqrtf(aq / (float)(packs_q * 8) + p.eps), rk = rsqrtf(ak / (float)((packs - packs_q) * 8) + p.eps);
+  T* q_out = static_cast<T*>(p.q_out) + t * p.H * p.stored;
+  const size_t page = slot >= 0 ? slot / p.page_size : 0, in_page = slot >= 0 ? slot % p.page_size : 0;
+  auto cache = [&](void* base, int g) { return static_cast<T*>(base) + ((page * p.G + g) * p.page_size + in_page) * p.stored; };
+  const bool tied = p.v.ptr == p.k.ptr && p.vdim == p.dim;      // the values are the k rows as they came
+#pragma unroll
+  for (int j = 0; j < JOINT_PACKS; ++j) {
+    const int i = threadIdx.x + j * blockDim.x;
+    if (i >= packs) continue;
+    const bool is_q = i < packs_q;
+    const int col = (is_q ? i : i - packs_q) * 8, head = col / p.dim, d = col - head * p.dim;
+    if (!is_q && slot < 0) continue;
+    if (!is_q && tied) store8<T>(cache(p.v_cache, head) + d, x[j]);
+    float w[8];
+    weight8(is_q ? p.qw : p.kw, col, w);
+    const float r = is_q ? rq : rk;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) x[j][e] *= r * w[e];
+    if (d < p.rot) turn_pairs8(x[j], p.cos, p.sin, angles + (d >> 1));
+    store8<T>((is_q ? q_out + (size_t)head * p.stored : cache(p.k_cache, head)) + d, x[j]);
+  }
+  const float zeros[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+  if (p.stored > p.dim) {
+    const int pad = (p.stored - p.dim) >> 3, heads = slot >= 0 ? p.H + p.G : p.H;
+    for (int i = threadIdx.x; i < heads * pad; i += blockDim.x) {
+      const int head = i / pad, d = p.dim + (i - head * pad) * 8;
+      store8<T>((head < p.H ? q_out + (size_t)head * p.stored : cache(p.k_cache, head - p.H)) + d, zeros);
+    }
+  }
+  if (slot < 0) return;
+  const int vper = p.stored >> 3, from = tied ? p.vdim >> 3 : 0, span = vper - from;
+  for (int i = threadIdx.x; i < p.G * span; i += blockDim.x) {
+    const int g = i / span, d = (from + i - g * span) * 8;
+    float y[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+    if (d < p.vdim) load8<T>(v + g * p.vdim + d, y);
+    store8<T>(cache(p.v_cache, g) + d, y);
   }
 }
 
@@ -687,13 +779,26 @@ TS_EXPORT int ts_gate_columns(const void* x, const void* gate, long long ldg, in
 TS_EXPORT int ts_joint_norm_kvwrite(int is_f32, const void* q, long long ldq, const void* k, long long ldk, const void* v,
                                     long long ldv, const void* qw, const void* kw, int w_is_f32, float eps, int H, int G,
                                     int dim, int vdim, int stored, void* q_out, void* k_cache, void* v_cache,
-                                    const int* slot_mapping, int page_size, int num_tokens, cudaStream_t stream) {
+                                    const int* slot_mapping, int page_size, int num_tokens, const float* cos, const float* sin,
+                                    const int* positions, int rot, int interleaved, cudaStream_t stream) {
   TS_REQUIRE(num_tokens > 0 && H > 0 && G > 0 && dim > 0 && vdim > 0 && stored >= dim && stored >= vdim,
              "joint_norm_kvwrite: sizes do not fit");
   TS_REQUIRE((qw == nullptr) == (kw == nullptr), "joint_norm_kvwrite: q and k are normed together or not at all");
   TS_REQUIRE(slot_mapping == nullptr || (k_cache && v_cache && page_size > 0), "joint_norm_kvwrite: no cache to write");
+  TS_REQUIRE(rot >= 0 && rot <= dim && rot % 2 == 0 && (rot == 0 || (cos && sin && positions)), "joint_norm_kvwrite: rotary size %d of %d", rot, dim);
   JointNorm p{Rows{q, ldq, is_f32}, Rows{k, ldk, is_f32}, Rows{v, ldv, is_f32}, VecParam{qw, w_is_f32},
-              VecParam{kw, w_is_f32}, eps, H, G, dim, vdim, stored, page_size, q_out, k_cache, v_cache, slot_mapping, is_f32};
+              VecParam{kw, w_is_f32}, eps, H, G, dim, vdim, stored, page_size, q_out, k_cache, v_cache, slot_mapping, is_f32,
+              cos, sin, positions, rot, interleaved};
+  const int packs = (H + G) * (dim / 8);
+  const uintptr_t all = (uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)qw | (uintptr_t)kw | (uintptr_t)q_out |
+                        (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)cos | (uintptr_t)sin;
+  if (qw && (interleaved || rot == 0) && ((dim | vdim | stored | rot) & 7) == 0 && ((ldq | ldk | ldv) & 7) == 0 && (all & 15) == 0 &&
+      packs <= JOINT_PACKS * JOINT_THREADS) {
+    const int threads = packs >= 512 ? 256 : (packs >= 128 ? 128 : (packs + 31) / 32 * 32);
+    if (is_f32) TS_LAUNCH("joint_norm_kvwrite", joint_norm_kvwrite_vec_kernel<float>, num_tokens, threads, 0, stream, p);
+    else TS_LAUNCH("joint_norm_kvwrite", joint_norm_kvwrite_vec_kernel<__nv_bfloat16>, num_tokens, threads, 0, stream, p);
+    return 0;
+  }
   TS_LAUNCH("joint_norm_kvwrite", joint_norm_kvwrite_kernel, num_tokens, H * dim >= 2048 ? 512 : (H * dim >= 512 ? 256 : 128), 0, stream, p);
   return 0;
 }

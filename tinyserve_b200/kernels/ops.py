@@ -16,6 +16,8 @@ from . import build
 #: u' = clamp(u, -bound, bound) it is g' sigmoid(1.702 g') (u' + 1)
 ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "bounded_swish": 2}
 BOUNDED_ACTIVATIONS = ("bounded_swish",)
+#: feed-forwards without a gate: act(x)
+PLAIN_ACTIVATIONS = {"relu_squared": 1}
 
 
 def activation_code(activation, limit=0.0):
@@ -383,9 +385,10 @@ def _tile_t(M):
     return 16 if M <= 16 else 32 if M <= 32 else 64 if M <= 64 else 128
 
 
-def _linear_tcgen05(x, weight, out_float32, splits=None, partials_only=False, scale=None, gated=0, bias=None, limit=0.0):
+def _linear_tcgen05(x, weight, out_float32, splits=None, partials_only=False, scale=None, gated=0, bias=None, limit=0.0, plain=0):
     """``scale``: the ScaledRows whose ``data`` is ``x``; ``gated``: activation code + 1 of the
-    gated epilogue (out [M, N / 2]); ``bias`` [N]: added in the epilogue (not with the others)."""
+    gated epilogue (out [M, N / 2]); ``bias`` [N]: added in the epilogue (not with the others); ``plain``: code
+    of an activation without a gate that the result passes there (with neither scale nor gate)."""
     M, K = x.shape
     N = weight.shape[0]
     out_cols = N // 2 if gated else N
@@ -405,6 +408,8 @@ def _linear_tcgen05(x, weight, out_float32, splits=None, partials_only=False, sc
     if scale is not None or gated:
         if bias is not None:
             raise ValueError("the scaled-rows and gated products take no bias")
+        if plain:
+            raise ValueError("the scaled-rows and gated products take no activation without a gate")
         _check(lib, lib.ts_gemm_tcgen05_fused(
             _ptr(x), _ptr(weight), _ptr(out), c_int(M), c_int(N), c_int(K), c_longlong(x.stride(0)),
             c_longlong(weight.stride(0)), c_longlong(out_cols), c_int(1 if out_float32 else 0), c_int(splits),
@@ -415,7 +420,7 @@ def _linear_tcgen05(x, weight, out_float32, splits=None, partials_only=False, sc
                                         c_longlong(x.stride(0)), c_longlong(weight.stride(0)), c_longlong(N),
                                         c_int(1 if out_float32 else 0), c_int(splits), _ptr(partials),
                                         _ptr(counters), _ptr(bias),
-                                        c_int(_vec_flag(bias, torch.bfloat16) if bias is not None else 0), _stream()))
+                                        c_int(_vec_flag(bias, torch.bfloat16) if bias is not None else 0), c_int(plain), _stream()))
     if partials_only:
         return SplitPartials(partials, splits, M, N, _tile_t(M), torch.bfloat16)
     return out
@@ -536,17 +541,22 @@ def _sequence():
     return build.load_unit("sequence.cu")
 
 
-def units_for(head_dims, key_dims=()) -> list:
-    """The (source, defines) units a model with these attention head sizes, and these key sizes of
-    its matrix-state mixers, needs."""
+def _streams():
+    return build.load_unit("streams.cu")
+
+
+def units_for(head_dims, key_dims=(), delta_dims=()) -> list:
+    """The (source, defines) units a model with these attention head sizes, these key sizes of
+    its matrix-state mixers and these of its delta-rule mixers needs."""
     units = [("elementwise.cu", {}), ("gemm_simt.cu", {}), ("gemm_tcgen05.cu", {}), ("gemm_pair_tcgen05.cu", {}),
-             ("sampler.cu", {}), ("latent_moe.cu", {}), ("sequence.cu", {})]
+             ("sampler.cu", {}), ("latent_moe.cu", {}), ("sequence.cu", {}), ("streams.cu", {})]
     units += [("attention_simt.cu", {"TS_HEAD_DIM": d}) for d in sorted(set(head_dims))]
     units += [("attention_mma.cu", _mma_defines(d)) for d in sorted(set(head_dims))
               if d <= MMA_MAX_HEAD_DIM]
     units += [("attention_tcgen05.cu", {"TS_HEAD_DIM": d}) for d in sorted(set(head_dims))
               if d in TCGEN05_HEAD_DIMS]
     units += [("linear_attention.cu", {"TS_KEY_DIM": d}) for d in sorted(set(key_dims))]
+    units += [("delta_rule.cu", {"TS_KEY_DIM": d}) for d in sorted(set(delta_dims))]
     return units
 
 
@@ -721,6 +731,28 @@ def gated_linear(x, weight, activation="silu", block=0, limit=0.0):
         return _linear_tcgen05(rows, weight, False, splits=1, gated=code + 1, limit=limit,
                                scale=x if rows is not x else None)
     return gated_activation(linear(x, weight), activation, block, limit)
+
+
+def plain_activation_(x, activation):
+    """x (contiguous, in place) <- act(x)."""
+    if activation not in PLAIN_ACTIVATIONS:
+        raise ValueError(f"unknown activation {activation!r} without a gate; known: {sorted(PLAIN_ACTIVATIONS)}")
+    _cuda(x)
+    if not x.is_contiguous():
+        raise TypeError("plain_activation_: x is contiguous")
+    lib = _elementwise()
+    _check(lib, lib.ts_plain_activation(c_int(_dt(x)), _ptr(x), c_longlong(x.numel()), c_int(PLAIN_ACTIVATIONS[activation]), _stream()))
+    return x
+
+
+def activated_linear(x, weight, activation):
+    """act(x @ weight^T) [M, N]: in the tcgen05 product's epilogue for up to TCGEN05_MAX_TOKENS bfloat16 rows,
+    else the product followed by the activation in place."""
+    x = materialize(x)
+    if x.dtype == torch.bfloat16 and weight.dtype == torch.bfloat16 and activation in PLAIN_ACTIVATIONS and _tcgen05_ok(x, weight):
+        _cuda(x, weight)
+        return _linear_tcgen05(x, weight, False, plain=PLAIN_ACTIVATIONS[activation])
+    return plain_activation_(linear(x, weight), activation)
 
 
 def qk_norm_rope_kvwrite(qkv, positions, num_heads, num_kv_heads, head_dim, rotary=None,
@@ -1864,12 +1896,14 @@ def gate_columns(attn, gate, vdim):
 
 
 def joint_norm_kvwrite(q, k, v, num_heads, num_kv_heads, dim, vdim, stored_dim, q_weight=None, k_weight=None, eps=0.0,
-                       k_cache=None, v_cache=None, slot_mapping=None, page_size=0):
+                       k_cache=None, v_cache=None, slot_mapping=None, page_size=0, rotary=None, positions=None):
     """q [T, H dim] and k [T, Hkv dim] each divided by the root mean square over the whole row (all
-    heads at once) and multiplied by a weight per column (both weights None: no norm); q goes to a
+    heads at once) and multiplied by a weight per column (both weights None: no norm), then rotated with
+    ``rotary`` (first ``rotary_dim`` elements of every head, at ``positions``); q goes to a
     [T, H, stored_dim] tensor (returned), k and v [T, Hkv vdim] to the cache slots of
-    ``slot_mapping`` (None: nothing is written), heads padded with zeros to ``stored_dim``."""
-    _cuda(q, k, v, q_weight, k_weight, k_cache, v_cache, slot_mapping)
+    ``slot_mapping`` (None: nothing is written), heads padded with zeros to ``stored_dim``.  v may be
+    the k rows themselves: they are stored as they come."""
+    _cuda(q, k, v, q_weight, k_weight, k_cache, v_cache, slot_mapping, positions if rotary is not None else None)
     T = q.shape[0]
     if q.shape[1] != num_heads * dim or k.shape[1] != num_kv_heads * dim or v.shape[1] != num_kv_heads * vdim:
         raise ValueError("joint_norm_kvwrite: q, k, v do not have heads x size columns")
@@ -1884,7 +1918,9 @@ def joint_norm_kvwrite(q, k, v, num_heads, num_kv_heads, dim, vdim, stored_dim, 
         c_int(_f32(q)), *_columns(q), *_columns(k), *_columns(v), _ptr(q_weight), _ptr(k_weight),
         c_int(_f32(q_weight) if q_weight is not None else 0), c_float(eps), c_int(num_heads), c_int(num_kv_heads),
         c_int(dim), c_int(vdim), c_int(stored_dim), _ptr(out), _ptr(k_cache), _ptr(v_cache), _ptr(slot_mapping),
-        c_int(page_size), c_int(T), _stream()))
+        c_int(page_size), c_int(T), _ptr(rotary.cos if rotary is not None else None),
+        _ptr(rotary.sin if rotary is not None else None), _ptr(positions if rotary is not None else None),
+        c_int(rotary.rotary_dim if rotary is not None else 0), c_int(int(rotary.interleaved) if rotary is not None else 0), _stream()))
     return out
 
 
@@ -2250,4 +2286,121 @@ def conv_heads_kvwrite(x, ctx, num_heads, num_kv_heads, dim, vdim, stored_dim, w
         _ptr(factor), c_int(_f32(factor) if factor is not None else 0), _ptr(state), _ptr(ctx.state_slots), _ptr(ctx.fresh),
         _ptr(ctx.cu_q), c_int(ctx.num_requests), c_int(max(1, min(ctx.max_q_len or T, T))), c_int(num_heads), c_int(G), c_int(dim),
         c_int(vdim), c_int(stored_dim), _ptr(out), _ptr(k_cache), _ptr(v_cache), _ptr(slot_mapping), c_int(page_size), _stream()))
+    return out
+
+
+# ----------------------------------------------------------------------------- several parallel residual streams
+MAX_STREAMS = 32
+
+
+class Streams:
+    """A residual of several streams per token.  Until a sub-layer's output has joined them all streams are the
+    one row they started from (``data`` [T, n], float32); from then on ``data`` is [T, count, n]."""
+
+    def __init__(self, start, count):
+        if start.dtype != torch.float32 or start.dim() != 2 or not start.is_contiguous():
+            raise TypeError("streams start from contiguous float32 rows")
+        self.data, self.count = start, int(count)
+        self.shape, self.device = (start.shape[0], start.shape[1]), start.device
+
+    @property
+    def apart(self):
+        return self.data.dim() == 3
+
+
+class StreamMix:
+    """A sub-layer's output on its way into the streams: x_t <- sum_s mix[s, t] x_s + out[t] y.  ``y``: a tensor
+    or an unfinished product (with its bias)."""
+
+    def __init__(self, y, mix, out):
+        self.y, self.mix, self.out = y, mix, out
+        self.shape, self.dtype, self.device = tuple(y.shape), y.dtype, y.device
+
+
+def stream_norm(x, streams, read, weight, eps, out_dtype, bias=None, centred=True, rows=None):
+    """``streams`` take in ``x`` (a StreamMix; None: they stay as they are), then u = sum_s read[s] x_s
+    (``read`` None: the plain sum) goes through a norm: (u - mean) / sqrt(var + eps) * weight (+ bias), or,
+    not ``centred``, the RMS norm.  With ``rows`` (int32) only those rows are read and returned, and
+    the streams are left as they are."""
+    S, (T, n) = streams.count, streams.shape
+    y = mix = out_w = y_bias = None
+    parts = _NO_PARTIALS
+    if x is not None:
+        y, mix, out_w = x.y, x.mix, x.out
+        if tuple(y.shape) != (T, n):
+            raise TypeError("stream_norm: the sub-layer's output does not have the streams' shape")
+        if isinstance(y, PendingProduct):
+            y_bias = y.bias
+            y = PendingProduct(y.x, y.weight, wide=y.wide).partials()
+        if isinstance(y, SplitPartials):
+            parts, y = y.args(), None
+        else:
+            y = materialize(y)
+            if y.dtype != out_dtype or not y.is_contiguous():
+                raise TypeError("stream_norm: the sub-layer's output is contiguous and of the compute dtype")
+        if mix.numel() != S * S or out_w.numel() != S or not mix.is_contiguous():
+            raise TypeError(f"stream_norm: coefficients of {S} streams")
+        if mix.dtype != out_w.dtype:
+            raise TypeError("stream_norm: coefficients of one dtype")
+    if read is not None and (read.numel() != S or (mix is not None and read.dtype != mix.dtype)):
+        raise TypeError(f"stream_norm: reading weights of {S} streams, of the coefficients' dtype")
+    _cuda(y, y_bias, mix, out_w, read, weight, bias, rows, streams.data)
+    src, dst = streams.data, None
+    if x is not None and rows is None:
+        dst = src if streams.apart else torch.empty(T, S, n, dtype=torch.float32, device=src.device)
+    num_out = T if rows is None else rows.shape[0]
+    h = torch.empty(num_out, n, dtype=out_dtype, device=src.device)
+    coef = mix if mix is not None else read
+    lib = _streams()
+    _check(lib, lib.ts_stream_mix(
+        c_int(_DTYPE[out_dtype]), _ptr(src), c_longlong(src.stride(0)), c_longlong(n if streams.apart else 0), _ptr(dst), _ptr(y), *parts,
+        _ptr(y_bias), c_int(_vec_flag(y_bias, out_dtype) if y_bias is not None else 0), _ptr(mix), _ptr(out_w), _ptr(read),
+        c_int(_vec_flag(coef, out_dtype) if coef is not None else 0), _ptr(weight), c_int(_vec_flag(weight, out_dtype)), _ptr(bias),
+        c_int(_vec_flag(bias, out_dtype) if bias is not None else 0), c_float(eps), c_int(1 if centred else 0), _ptr(h), _ptr(rows),
+        c_int(num_out), c_int(n), c_int(S), _stream()))
+    if dst is not None:
+        streams.data = dst
+    return h
+
+
+# ----------------------------------------------------------------------------- gated delta rule
+DELTA_MAX_KEY_DIM = 1024
+#: requests of up to this many tokens in a step run the wide form of the kernel (the state's transfer counts), longer
+#: portions the narrow one in tiles of DELTA_TILE value columns (the chain from token to token counts)
+DELTA_WIDE_MAX_TOKENS = 4
+DELTA_TILE = 16
+
+
+def delta_rule(q, k, v, gate, logits, bias, rate, state, ctx, num_heads, key_dim, value_dim, norm_weight, eps, out_dtype,
+               q_scale=1.0, qk_group=1, tile=None):
+    """Per request and head S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q over this step's tokens, from
+    and to ``state`` [slots, H, key_dim, value_dim] (float32); returns [T, H value_dim] = o / rms(o) * norm_weight *
+    silu(gate).  q, k [T, H / qk_group key_dim] are made unit vectors per head (q then times ``q_scale``); logits
+    float32 [T, 2 H] hold a and b: g = exp(-exp(rate) softplus(a + bias)), beta = sigmoid(b).  The operands may
+    be column ranges.  ``tile``: value columns of a block (0: the wide form; None: by the step's longest portion)."""
+    _cuda(q, k, v, gate, logits, bias, rate, state, norm_weight)
+    T, H = q.shape[0], num_heads
+    if H % qk_group or q.shape[1] != H // qk_group * key_dim or k.shape != q.shape or v.shape[1] != H * value_dim or gate.shape != v.shape:
+        raise ValueError("delta_rule: q, k, v, gate do not have heads x size columns")
+    if logits.dtype != torch.float32 or tuple(logits.shape) != (T, 2 * H) or logits.stride(1) != 1:
+        raise TypeError("delta_rule: the logits are float32 [T, 2 heads]")
+    if state.dtype != torch.float32 or tuple(state.shape[1:]) != (H, key_dim, value_dim) or not state.is_contiguous():
+        raise TypeError("delta_rule: the state is contiguous float32 [slots, H, key_dim, value_dim]")
+    if bias.numel() != H or rate.numel() != H or norm_weight.numel() != value_dim:
+        raise TypeError("delta_rule: a bias and a rate per head, a norm weight per value column")
+    if not 0 < key_dim <= DELTA_MAX_KEY_DIM:
+        raise ValueError(f"delta_rule: key sizes of up to {DELTA_MAX_KEY_DIM}")
+    longest = max(1, min(getattr(ctx, "max_q_len", 0) or T, T))
+    if tile is None:
+        tile = 0 if longest <= DELTA_WIDE_MAX_TOKENS else DELTA_TILE
+    lib = build.load_unit("delta_rule.cu", {"TS_KEY_DIM": key_dim})
+    spread = lib.ts_delta_rule_column_tiles(c_int(value_dim), c_int(tile)) > 1
+    raw = torch.empty(T, H * value_dim, dtype=torch.float32, device=q.device) if spread else None
+    out = torch.empty(T, H * value_dim, dtype=out_dtype, device=q.device)
+    _check(lib, lib.ts_delta_rule(
+        c_int(_dt(q)), *_columns(q), *_columns(k), *_columns(v), *_columns(gate), _ptr(logits), c_longlong(logits.stride(0)), _ptr(bias),
+        c_int(_f32(bias)), _ptr(rate), c_int(_f32(rate)), c_float(q_scale), _ptr(state), _ptr(ctx.state_slots), _ptr(ctx.fresh),
+        _ptr(ctx.cu_q), c_int(ctx.num_requests), c_int(longest), c_int(T), _ptr(norm_weight), c_int(_f32(norm_weight)), c_float(eps),
+        _ptr(out), c_longlong(out.stride(0)), _ptr(raw), c_int(H), c_int(value_dim), c_int(qk_group), c_int(tile), _stream()),
+        2 if spread else 1)
     return out

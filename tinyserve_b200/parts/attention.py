@@ -20,12 +20,14 @@ With a window, ``keep_first`` > 0 keeps the first tokens of every sequence visib
 queries (they keep their own positions, and their pages are never released).
 
 Further forms, each a parameter: ``joint_norm`` (q and k each divided by the root mean square over
-all their heads at once, before they are split into heads, with one weight per column, plain);
+all their heads at once, before they are split into heads and rotated, with one weight per column, plain);
 ``chunk`` > 0 (position i sees j <= i only if i // chunk == j // chunk, chunks counted from
 position 0 of the sequence); ``distance_slopes`` (one slope per head: slope * (i - j) is taken off
 the scaled score); ``sinks`` (a learned number per head whose exponential joins the softmax sum,
 without key or value); ``out_gate`` (the concatenated heads times sigmoid(W_g h), element by
-element, before the output projection).  Biases on q, k and v go with all of them.
+element, before the output projection).  Biases on q, k and v go with all of them, and ``out_bias`` adds one
+to the output projection.  ``tied_values``: there is no value projection, a key head as projected (bias
+included, before norm and rotation) is also the value head.
 
 ``softcap`` c > 0: the scaled score s becomes c tanh(s / c) before the softmax.
 
@@ -66,7 +68,7 @@ class Attention(Mixer):
                  position=None, window=0, scale=None, names=None, value_dim=None, unit_norm_eps=None,
                  head_gate=False, keep_first=0, joint_norm=False, norm_eps=0.0, chunk=0, distance_slopes=None,
                  sinks=False, out_gate=False, softcap=0.0, differential=None, conv_taps=0, query_factor=False,
-                 sink_score=None, value_rotation=None, borrows_kv=False):
+                 sink_score=None, value_rotation=None, borrows_kv=False, out_bias=False, tied_values=False):
         super().__init__()
         self.names = dict(DEFAULT_NAMES, **(names or {}))
         if num_heads % num_kv_heads:
@@ -119,15 +121,17 @@ class Attention(Mixer):
                              "slopes, learned sinks, output gate or a second map")
         if further and (self.differential or (self.has_sinks and self.sink_score is not None)):
             raise ValueError("attention: two score maps come alone, and a sink is learned or constant")
-        self.general = (further or self.value_dim != head_dim or self.unit_norm_eps is not None or self.head_gate
+        self.out_bias, self.tied_values = bool(out_bias), bool(tied_values)
+        if self.tied_values and (self.value_dim != head_dim or self.borrows_kv or self.convolved or self.differential or self.value_rotation is not None):
+            raise ValueError("attention: values that are the keys have the keys' head size and come without a convolution, another "
+                             "layer's cache, a second map and turned values")
+        self.general = (further or self.tied_values or self.value_dim != head_dim or self.unit_norm_eps is not None or self.head_gate
                         or self.keep_first > 0 or extended or self.softcap > 0 or self.maps > 1)
-        if self.general and ((qk_norm is not None and (extended or self.unit_norm_eps is not None))
-                             or (bias and not extended)):
+        if self.general and qk_norm is not None and (extended or self.unit_norm_eps is not None):
             raise ValueError("attention: the unit norm and the forms with a joint norm, chunks, slopes, sinks or an output "
-                             "gate come without a weighted per-head q/k norm; a value size of its own, the unit norm and "
-                             "the head gate come without biases")
-        if self.joint_norm and (self.unit_norm_eps is not None or position is not None):
-            raise ValueError("attention: the norm over all heads comes without rotation and without the unit norm")
+                             "gate come without a weighted per-head q/k norm")
+        if self.joint_norm and self.unit_norm_eps is not None:
+            raise ValueError("attention: the norm over all heads comes without the unit norm")
         self.slopes = self.sinks = None
         widest = max(head_dim, self.value_dim)
         self.stored_dim = -(-widest // 16) * 16 if self.general else head_dim
@@ -136,6 +140,8 @@ class Attention(Mixer):
         self.v_size = num_kv_heads * self.value_dim
         if self.borrows_kv:
             self.kv_size = self.v_size = 0
+        if self.tied_values:
+            self.v_size = 0
         self.map_factor = None       # lambda of the two maps, made when the tensors are bound
         self.gate_size = num_heads if self.head_gate else (num_heads * self.value_dim if self.out_gate else 0)
 
@@ -153,8 +159,8 @@ class Attention(Mixer):
         q, kv, vs = self.q_size, self.kv_size, self.v_size
         nm = self.names
         rows = ((nm["q"], 0, q), (nm["k"], q, q + kv), (nm["v"], q + kv, q + kv + vs))
-        if self.borrows_kv:
-            rows = rows[:1]
+        if self.borrows_kv or self.tied_values:
+            rows = rows[:1 if self.borrows_kv else 2]
         qkv_rows = rows
         if self.gate_size:
             rows += ((nm["gate"], q + kv + vs, q + kv + vs + self.gate_size),)
@@ -169,6 +175,9 @@ class Attention(Mixer):
             # (the gate's rows, where there are any, have no bias: ``bind`` zeroes theirs)
             specs["qkv_proj.bias"] = ParamSpec((q + kv + vs + self.gate_size,), role="matrix", init="normal", sources=tuple(
                 Source(f"{n}.bias", a, b) for n, a, b in qkv_rows))
+        if self.out_bias:
+            specs["o_proj.bias"] = ParamSpec((self.hidden_size,), role="matrix", init="normal",
+                                             sources=(Source(f"{nm['o']}.bias", 0, self.hidden_size),))
         if self.joint_norm:
             specs["q_norm.weight"] = ParamSpec((q,), role="vector", init="norm_weight",
                                                sources=(Source(f"{nm['q_norm']}.weight", 0, q),))
@@ -247,6 +256,8 @@ class Attention(Mixer):
         v_end = k_end + self.v_size
         slots = view.slot_mapping if call.writes_cache and not self.borrows_kv else None
         k, v = (None, None) if self.borrows_kv else (qkv[:, q_end:k_end], qkv[:, k_end:v_end])
+        if self.tied_values:
+            v = k
         if self.convolved:
             return ops.conv_heads_kvwrite(
                 qkv[:, :v_end], ctx, self.num_heads, self.num_kv_heads, self.head_dim, self.value_dim, self.stored_dim,
@@ -256,7 +267,8 @@ class Attention(Mixer):
             return ops.joint_norm_kvwrite(
                 qkv[:, :q_end], k, v, self.num_heads, self.num_kv_heads, self.head_dim,
                 self.value_dim, self.stored_dim, self.w.get("q_norm.weight"), self.w.get("k_norm.weight"), self.norm_eps,
-                k_cache=cache.k, v_cache=cache.v, slot_mapping=slots, page_size=view.page_size)
+                k_cache=cache.k, v_cache=cache.v, slot_mapping=slots, page_size=view.page_size, rotary=self.position,
+                positions=ctx.positions)
         M = self.maps
         return ops.rope_unit_kvwrite(
             qkv[:, :q_end], k, v, ctx.positions, self.num_heads * M,
@@ -287,7 +299,7 @@ class Attention(Mixer):
             out = ops.head_gate(out, qkv[:, v_end:] if self.head_gate else None, self.value_dim)
         else:
             out = out.view(out.shape[0], self.num_heads * self.value_dim)
-        return ops.linear(out, self.w["o_proj.weight"], allow_pending=True)
+        return ops.linear(out, self.w["o_proj.weight"], self.w.get("o_proj.bias"), allow_pending=True)
 
     def _forward_general(self, h, ctx, call):
         return self.forward_projected([ops.linear(h, self.w["qkv_proj.weight"], self.w.get("qkv_proj.bias"))], h, ctx, call)
@@ -304,7 +316,7 @@ class Attention(Mixer):
             self.k_norm.w["weight"] if self.k_norm is not None else None,
             self.q_norm.eps if self.q_norm is not None else 0.0,
             cache.k, cache.v, view, ctx, self.scale, self.window, write_cache=call.writes_cache)
-        return ops.linear(out.view(out.shape[0], self.q_size), self.w["o_proj.weight"], allow_pending=True)
+        return ops.linear(out.view(out.shape[0], self.q_size), self.w["o_proj.weight"], self.w.get("o_proj.bias"), allow_pending=True)
 
 
 register_mixer("attention", Attention)

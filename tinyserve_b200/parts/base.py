@@ -35,7 +35,7 @@ class ParamSpec:
     tensor that the checkpoint stores in 32-bit stays 32-bit.
     role "int_table": integer table, kept as int32.
     init: "normal" (N(0, 0.02)), "norm_weight" (1 + U(-0.1, 0.1)), "around_zero" (U(-0.1, 0.1)), "wide" (N(0, 1)),
-    "unit_interval" (U(0.05, 0.95)) or "zeros", used by the random-weights mode.  ``sources`` lists the checkpoint tensors that fill it
+    "unit_interval" (U(0.05, 0.95)), "near_identity" (a square matrix, 1 on the diagonal, + U(-0.1, 0.1)) or "zeros", used by the random-weights mode.  ``sources`` lists the checkpoint tensors that fill it
     (default: one tensor of the same name and shape).  ``interleave_halves`` = b > 0: after the
     sources are placed, the rows of the first and the second half alternate in blocks of b rows
     (first-half rows [0, b), second-half rows [0, b), first-half rows [b, 2b), ...).
@@ -161,6 +161,12 @@ class Norm(Part):
 
     def rms_parameters(self):
         """(weight, eps) if this norm is a plain RMSNorm, else None."""
+        return None
+
+    def row_parameters(self):
+        """(weight, bias or None, eps, centred) if this norm divides a row by its root mean square (``centred``:
+        of the deviations from its mean) and applies weight and bias, else None: the kernels that run it
+        right behind something else."""
         return None
 
 

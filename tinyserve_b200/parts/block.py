@@ -15,7 +15,7 @@ from __future__ import annotations
 
 from ..config.model_config import LayerSpec
 from ..kernels import ops
-from .base import ParamSpec, Part, StateSpec, build_feed_forward, build_mixer, build_norm
+from .base import Norm, ParamSpec, Part, StateSpec, build_feed_forward, build_mixer, build_norm
 
 
 def add_and_norm(norm, x, residual, reader=None, rows=None, compute_dtype=None):
@@ -23,7 +23,9 @@ def add_and_norm(norm, x, residual, reader=None, rows=None, compute_dtype=None):
     mixer or feed-forward returned: a tensor or one of ops' unfinished products.  A plain RMSNorm
     goes to the fused kernels, and a reader that only multiplies its input by a matrix
     (``accepts_scaled_rows``) may get rows without their norm factor; any other norm gets a
-    finished tensor."""
+    finished tensor.  ``residual`` may be an ``ops.Streams``: the norm then reads the sum of the streams."""
+    if isinstance(residual, ops.Streams):
+        return _stream_norm(norm, x, residual, None, rows, compute_dtype)
     rms = norm.rms_parameters()
     if isinstance(x, ops.NormedAddend) and rms is not None:
         # the norm on the sub-layer's output, the add and this norm are one kernel
@@ -34,6 +36,13 @@ def add_and_norm(norm, x, residual, reader=None, rows=None, compute_dtype=None):
     scaled_ok = rows is None and reader is not None and getattr(reader, "accepts_scaled_rows", False)
     return ops.add_rmsnorm(x, residual, weight, eps, compute_dtype or residual_compute_dtype(norm, x),
                            rows=rows, scaled_ok=scaled_ok)
+
+
+def _stream_norm(norm, x, streams, read, rows, compute_dtype):
+    """What lies between two sub-layers of a block of several streams, in one kernel: the streams take in x (None
+    or an ``ops.StreamMix``), the next sub-layer reads them with ``read`` (None: their sum), through its norm."""
+    weight, bias, eps, centred = norm.row_parameters()
+    return ops.stream_norm(x, streams, read, weight, eps, compute_dtype, bias=bias, centred=centred, rows=rows)
 
 
 def residual_compute_dtype(norm, x):
@@ -286,8 +295,65 @@ class PostNormBlock(Part):
         return None
 
 
+class HyperConnectionBlock(Part):
+    """Pre-norm sub-layers on several parallel streams x_1 .. x_s (``LayerSpec.options["streams"]``): a sub-layer
+    reads u = sum_s in[s] x_s through its norm, and its output y joins all of them at once,
+    x_t <- sum_s mix[s, t] x_s + out[t] y (mix is indexed [from, to]); in, mix and out are learned, for each of the two
+    sub-layers.  The model keeps the streams (``ModelSpec.streams``); the block hands on its last output with
+    its coefficients (``ops.StreamMix``) and the kernel of the next norm brings the streams up to date.  A layer
+    without a feed-forward (``LayerSpec.ffn`` None) has the first sub-layer only."""
+    capturable = True
+
+    def __init__(self, spec: LayerSpec, hidden_size: int):
+        super().__init__()
+        self.streams = int(spec.options.get("streams", 0))
+        if not 1 <= self.streams <= ops.MAX_STREAMS:
+            raise ValueError(f"hyper-connections: 1 to {ops.MAX_STREAMS} streams, got {self.streams}")
+        self.mixer = build_mixer(spec.mixer)
+        self.ffn = build_feed_forward(spec.ffn) if spec.ffn is not None else None
+        self.input_norm = build_norm(spec.norm, hidden_size)
+        self.ffn_norm = build_norm(spec.norm, hidden_size) if self.ffn is not None else None
+        for norm in (self.input_norm, self.ffn_norm):
+            if norm is not None and type(norm).row_parameters is Norm.row_parameters:
+                raise ValueError("hyper-connections: norms that the streams' kernel can run (layernorm, rmsnorm)")
+        self._names = {"mixer": spec.name_of("mixer", self.mixer.tree_name),
+                       "ffn": spec.name_of("ffn", self.ffn.tree_name if self.ffn is not None else ""),
+                       "input_norm": spec.name_of("input_norm"), "ffn_norm": spec.name_of("ffn_norm", "ffn_norm"),
+                       "mixer_streams": spec.name_of("mixer_streams", "mixer_streams"),
+                       "ffn_streams": spec.name_of("ffn_streams", "ffn_streams")}
+
+    def children(self):
+        n = self._names
+        out = {n["mixer"]: self.mixer, n["input_norm"]: self.input_norm}
+        if self.ffn is not None:
+            out.update({n["ffn"]: self.ffn, n["ffn_norm"]: self.ffn_norm})
+        return out
+
+    def param_specs(self):
+        specs, s = {}, self.streams
+        for which in ("mixer_streams", "ffn_streams") if self.ffn is not None else ("mixer_streams",):
+            name = self._names[which]
+            specs[f"{name}.in"] = ParamSpec((s,), role="vector", init="norm_weight")
+            specs[f"{name}.out"] = ParamSpec((s,), role="vector", init="norm_weight")
+            specs[f"{name}.mix"] = ParamSpec((s, s), role="vector", init="near_identity")
+        return specs
+
+    def _read(self, norm, which, x, streams, ctx):
+        return _stream_norm(norm, x, streams, self.w[f"{self._names[which]}.in"], None, ctx.dtype)
+
+    def _join(self, y, which):
+        name = self._names[which]
+        return ops.StreamMix(y, self.w[f"{name}.mix"], self.w[f"{name}.out"])
+
+    def forward(self, x, residual, ctx, call):
+        x = self._join(self.mixer.forward(self._read(self.input_norm, "mixer_streams", x, residual, ctx), ctx, call), "mixer_streams")
+        if self.ffn is None:
+            return x
+        return self._join(self.ffn.forward(self._read(self.ffn_norm, "ffn_streams", x, residual, ctx), ctx), "ffn_streams")
+
+
 ARRANGEMENTS = {"pre_norm": PreNormBlock, "parallel": ParallelBlock, "parallel_two_norms": ParallelTwoNormsBlock, "sandwich": SandwichBlock,
-                "post_norm": PostNormBlock}
+                "post_norm": PostNormBlock, "hyper_connections": HyperConnectionBlock}
 
 
 def build_block(spec: LayerSpec, hidden_size: int):

@@ -29,6 +29,12 @@ the value size, silu gate, output projection) is ``MatrixStateMixer``; they diff
   dt = softplus(dt + bias), S_t = exp(-exp(A_log) dt) S_(t-1) + dt B_t x_t^T, y_t = S_t^T C_t + D x_t;
   y silu(z) is RMS-normed in groups over all heads.  B plays k, C plays q, shared by the heads of a group.
 
+* ``GatedDeltaRule``: the state is corrected, not only added to: S <- g S; u = beta (v - S^T k); S <- S + k u^T;
+  o = S^T q.  q, k, v pass a short causal convolution and silu; q and k become unit vectors per head (q times
+  key_dim^(-1/2)) and are shared by groups of heads; per head and token g = exp(-exp(A) softplus(W_a h + bias)) and
+  beta = sigmoid(W_b h); the head's output is RMS-normed with one weight of value size for all heads, times silu(W_g h)
+  (csrc/delta_rule.cu).
+
 Everything behind the projections is 32-bit (angles, decays, gates, step sizes, state, output norm):
 csrc/linear_attention.cu.  The decay logits z leave their product in 32-bit."""
 from __future__ import annotations
@@ -318,6 +324,66 @@ class Mamba2(Mixer):
         return ops.linear(out, self.w["o_proj.weight"], allow_pending=True)
 
 
+class GatedDeltaRule(Mixer):
+    tree_name = "mixer"
+    capturable = True
+
+    def __init__(self, hidden_size, num_heads, num_kv_heads, key_dim, value_dim, conv_taps, eps, names=None):
+        super().__init__()
+        self.names = dict({"q": "q", "k": "k", "v": "v", "g": "g", "o": "o", "a": "a", "b": "b", "conv": "{name}.conv",
+                           "dt_bias": "dt_bias", "a_log": "A_log", "norm": "norm"}, **(names or {}))
+        self.hidden_size, self.num_heads, self.num_kv_heads = hidden_size, int(num_heads), int(num_kv_heads)
+        self.key_dim, self.value_dim, self.taps, self.eps = int(key_dim), int(value_dim), int(conv_taps), float(eps)
+        if self.num_kv_heads < 1 or self.num_heads % self.num_kv_heads:
+            raise ValueError(f"delta rule: {num_heads} heads do not share {num_kv_heads} query/key heads evenly")
+        if not 0 < self.key_dim <= ops.DELTA_MAX_KEY_DIM or self.value_dim < 1:
+            raise ValueError(f"delta rule: key size {key_dim} (up to {ops.DELTA_MAX_KEY_DIM}) or value size {value_dim} is not supported")
+        if not 1 <= self.taps <= ops.CAUSAL_CONV_MAX_TAPS:
+            raise ValueError(f"delta rule: a convolution of 1 to {ops.CAUSAL_CONV_MAX_TAPS} taps, got {conv_taps}")
+        self.qk_size, self.v_size = self.num_kv_heads * self.key_dim, self.num_heads * self.value_dim
+        self.conv_channels = 2 * self.qk_size + self.v_size
+
+    def param_specs(self):
+        nm, qk, v, n, H = self.names, self.qk_size, self.v_size, self.hidden_size, self.num_heads
+        rows = ((nm["q"], 0, qk), (nm["k"], qk, 2 * qk), (nm["v"], 2 * qk, 2 * qk + v))
+        return {
+            "in_proj.weight": ParamSpec((self.conv_channels + v, n), sources=tuple(Source(f"{name}.weight", a, b) for name, a, b in rows)
+                                        + (Source(f"{nm['g']}.weight", self.conv_channels, self.conv_channels + v),)),
+            # decay and write strength enter the recurrence: their product leaves in 32-bit
+            "gates.weight": ParamSpec((2 * H, n), sources=(Source(f"{nm['a']}.weight", 0, H), Source(f"{nm['b']}.weight", H, 2 * H))),
+            "conv.weight": ParamSpec((self.conv_channels, self.taps), init="wide", sources=tuple(
+                Source(nm["conv"].format(name=name) + ".weight", a, b) for name, a, b in rows)),
+            "dt_bias": ParamSpec((H,), role="vector", init="wide", sources=(Source(nm["dt_bias"], 0, H),)),
+            "a_log": ParamSpec((H,), role="vector", init="wide", sources=(Source(nm["a_log"], 0, H),)),
+            "norm.weight": ParamSpec((self.value_dim,), role="vector", init="norm_weight",
+                                     sources=(Source(f"{nm['norm']}.weight", 0, self.value_dim),)),
+            "o_proj.weight": ParamSpec((n, v), sources=(Source(f"{nm['o']}.weight", 0, n),)),
+        }
+
+    def state_specs(self):
+        specs = {"": StateSpec((self.num_heads, self.key_dim, self.value_dim), "float32")}
+        if self.taps > 1:
+            specs["conv"] = StateSpec((self.taps - 1, self.conv_channels), "float32")
+        return specs
+
+    def input_products(self):
+        return [ops.InputProduct(self.w["in_proj.weight"]), ops.InputProduct(self.w["gates.weight"], None, True)]
+
+    def forward_projected(self, projected, h, ctx, call):
+        proj, logits = ops.materialize(projected[0]), projected[1]
+        qk, C = self.qk_size, self.conv_channels
+        x = ops.causal_conv(proj[:, :C], self.w["conv.weight"], ctx.state(call.state_of("conv")) if self.taps > 1 else None, ctx,
+                            ctx.dtype, activation="silu")
+        out = ops.delta_rule(x[:, :qk], x[:, qk:2 * qk], x[:, 2 * qk:], proj[:, C:], logits, self.w["dt_bias"], self.w["a_log"],
+                             ctx.state(call.state_of("")), ctx, self.num_heads, self.key_dim, self.value_dim, self.w["norm.weight"],
+                             self.eps, ctx.dtype, q_scale=self.key_dim ** -0.5, qk_group=self.num_heads // self.num_kv_heads)
+        return ops.linear(out, self.w["o_proj.weight"], allow_pending=True)
+
+    def forward(self, h, ctx, call):
+        return self.forward_projected(ops.linear_beside([(h, self.input_products())])[0], h, ctx, call)
+
+
+register_mixer("gated_delta_rule", GatedDeltaRule)
 register_mixer("hgrn2", HGRN2)
 register_mixer("mlstm", MLSTM)
 register_mixer("mamba2", Mamba2)

@@ -8,6 +8,8 @@ layout where the product is someone else's.
 polynomial of normed powers, c0 N(z) + c1 N(z^2) + c2 N(z^3) + c3 with four learned numbers and N(y) =
 y / sqrt(mean(y^2) + eps) over a token's whole row (``ops.poly_norm``).
 
+``PlainMLP`` has neither gate nor biases: down(act(up(x))), act the square of relu.
+
 ``activation`` "bounded_swish" with ``limit`` L: g = min(gate(x), L), u = clamp(up(x), -L, L),
 down(g sigmoid(1.702 g) (u + 1))."""
 from __future__ import annotations
@@ -84,3 +86,28 @@ class PolyNormMLP(FeedForward):
 
 
 register_feed_forward("poly_norm_mlp", PolyNormMLP)
+
+
+class PlainMLP(FeedForward):
+    tree_name = "mlp"
+    capturable = True
+    accepts_scaled_rows = True
+
+    def __init__(self, hidden_size, intermediate_size, activation="relu_squared", names=None):
+        super().__init__()
+        self.names = dict(DEFAULT_NAMES, **(names or {}))
+        self.hidden_size, self.intermediate_size, self.activation = hidden_size, intermediate_size, activation
+        if activation not in ops.PLAIN_ACTIVATIONS:
+            raise ValueError(f"unknown activation {activation!r} without a gate; known: {sorted(ops.PLAIN_ACTIVATIONS)}")
+
+    def param_specs(self):
+        i, n, nm = self.intermediate_size, self.hidden_size, self.names
+        return {"up_proj.weight": ParamSpec((i, n), sources=(Source(f"{nm['up']}.weight", 0, i),)),
+                "down_proj.weight": ParamSpec((n, i), sources=(Source(f"{nm['down']}.weight", 0, n),))}
+
+    def forward(self, h, ctx):
+        return ops.linear(ops.activated_linear(h, self.w["up_proj.weight"], self.activation), self.w["down_proj.weight"],
+                          allow_pending=True)
+
+
+register_feed_forward("plain_mlp", PlainMLP)

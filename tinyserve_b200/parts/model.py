@@ -100,6 +100,8 @@ class DecoderModel(Part):
             self.lm_head.set_path(spec.name_of("lm_head"))
         if self.embed_position is not None:
             self.embed_position.set_path(spec.name_of("embed_position"))
+        if any(layer.options.get("streams", 0) != spec.streams for layer in spec.layers) or (spec.streams and self.stream_ops):
+            raise ValueError(f"{spec.streams} residual streams: every layer keeps as many, and nothing runs between layers")
         self._resolve_order()
         #: every part allows a captured graph of its forward pass to be replayed
         self.capturable = all(part.capturable for part in self.named_parts())
@@ -175,6 +177,8 @@ class DecoderModel(Part):
         if self.embed_position is not None:
             self.embed_position.add_to_embeddings(residual, ctx)
         first = residual.clone() if any(op.needs_first for op in self.stream_ops.values()) else None
+        if self.spec.streams:
+            residual = ops.Streams(residual, self.spec.streams)
         x = None
         for call in self.calls:
             for op, arg in call.before:

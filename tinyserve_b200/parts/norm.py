@@ -40,6 +40,9 @@ class RMSNorm(Norm):
     def rms_parameters(self):
         return self.w["weight"], self.eps
 
+    def row_parameters(self):
+        return self.w["weight"], None, self.eps, False
+
 
 register_norm("rmsnorm", RMSNorm)
 
@@ -72,6 +75,9 @@ class LayerNorm(Norm):
     def add_forward(self, x, residual, rows=None):
         return ops.add_layernorm(x, residual, self.w["weight"], self.eps, self.compute_dtype,
                                  bias=self.w.get("bias"), rows=rows)
+
+    def row_parameters(self):
+        return self.w["weight"], self.w.get("bias"), self.eps, True
 
 
 register_norm("layernorm", LayerNorm)
