@@ -202,3 +202,19 @@ def forward(cfg, W, tokens, keep_layers=False):
         after.append(X.sum(0))
     logits = centred_norm(X.sum(0), W["final.norm"], eps) @ W["embed"].T
     return (logits, torch.stack(after)) if keep_layers else logits
+
+
+def logits(cfg, W, tokens):
+    with torch.no_grad():
+        return forward(cfg, W, tokens)
+
+
+def greedy(cfg, W, prompt, count):
+    """``count`` greedy tokens, and by how much each led the second best."""
+    ids, out, gaps = list(prompt), [], []
+    for _ in range(count):
+        top = logits(cfg, W, ids)[-1].topk(2)
+        out.append(int(top.indices[0]))
+        gaps.append(float(top.values[0] - top.values[1]))
+        ids.append(out[-1])
+    return out, gaps

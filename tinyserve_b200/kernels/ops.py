@@ -125,6 +125,11 @@ def raise_on_device_error() -> None:
                           "the access was skipped and the engine stops")
 
 
+class _HeldPointer(c_void_p):
+    """A pointer that keeps its tensor: whoever holds the arguments of a launch that has not happened yet
+    holds the memory, which could otherwise be handed out again as the launch's own output."""
+
+
 class SplitPartials:
     """The result of a matrix product as split-K partial tiles: the product's kernel stopped
     before adding them up, because the next kernel (residual add + norm, or the q/k norm + rotary
@@ -138,8 +143,9 @@ class SplitPartials:
         self.device = data.device
 
     def args(self):
-        return (_ptr(self.data), c_int(self.splits), c_int(self.n_tiles), c_int(self.t_tiles),
-                c_int(self.tile_t))
+        pointer = _HeldPointer(self.data.data_ptr())
+        pointer.held = self.data
+        return (pointer, c_int(self.splits), c_int(self.n_tiles), c_int(self.t_tiles), c_int(self.tile_t))
 
     def materialize(self):
         out = torch.empty(self.M, self.N, dtype=self.dtype, device=self.device)

@@ -12,7 +12,7 @@ Beyond that model: values may have a head size of their own (``value_dim``); q a
 divided by their root mean square per head, without a weight, after the position encoding
 (``unit_norm_eps``); every head's output may be multiplied by sigmoid of one number per head, a
 projection of the same input (``head_gate``, rows of the fused projection after v).  With any
-of these the heads are stored ``stored_dim`` wide (the larger of the two head sizes, rounded up
+of these, and where the head size is no multiple of 16, the heads are stored ``stored_dim`` wide (the larger of the two head sizes, rounded up
 to what the attention kernels take), padded with zeros: zero key columns add nothing to a score
 and the padded output columns are dropped.
 
@@ -126,7 +126,7 @@ class Attention(Mixer):
             raise ValueError("attention: values that are the keys have the keys' head size and come without a convolution, another "
                              "layer's cache, a second map and turned values")
         self.general = (further or self.tied_values or self.value_dim != head_dim or self.unit_norm_eps is not None or self.head_gate
-                        or self.keep_first > 0 or extended or self.softcap > 0 or self.maps > 1)
+                        or self.keep_first > 0 or extended or self.softcap > 0 or self.maps > 1 or head_dim % 16 != 0)
         if self.general and qk_norm is not None and (extended or self.unit_norm_eps is not None):
             raise ValueError("attention: the unit norm and the forms with a joint norm, chunks, slopes, sinks or an output "
                              "gate come without a weighted per-head q/k norm")
