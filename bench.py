@@ -35,6 +35,11 @@ feed-forwards, dense and as experts, a repeated group of layers) beside Delilorn
 measures Gunulorn (mixer and feed-forward side by side on two norms, convolved attention, window attention
 over turned values, a polynomial of normed powers, experts beside identity experts) beside Babadra, the
 closest design (dense and gated-expert feed-forwards in turn, grouped-query attention).
+
+    python bench.py --arch ronolorn [--sizes 2048,4096]
+
+measures Ronolorn (a memory under the gated delta rule, window attention with and without a value projection, four
+parallel residual streams) beside Dudatar, the closest design (gated linear attention, attention, dense feed-forwards).
 """
 from __future__ import annotations
 
@@ -459,6 +464,25 @@ def gunulorn_shapes(width):
     gunulorn = {"architecture": "Gunulorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_scale": 0.5,
                 "logit_softcap": 30.0, "layers": [{"type": "attention", "mixer": conv, "mlp": dense}, turned, reader, turned, reader, turned]}
     return gunulorn, babadra
+
+
+def ronolorn_shapes(width):
+    """A Ronolorn of real layer sizes at ``width``: a delta-rule memory, window attention, window attention whose
+    values are its keys, twice: six blocks on four streams.  As many heads of 128 as the Dudatar of the same width
+    has, memories of 128 x 128 for as many heads on half as many query/key heads, windows of 1,024 keys, dense
+    feed-forwards of two matrices with as many weights as Dudatar's three."""
+    dudatar, _ = dudatar_shapes(width)
+    heads, vocab = width // 128, 32768
+    mlp = {"kind": "dense", "ff": dudatar["layers"][0]["mlp"]["ff"] * 3 // 2}
+    base = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 1024}}
+    delta = {"heads": heads, "kv_heads": heads // 2, "dim": 128, "vdim": 128, "conv": 4}
+    scaling = {"factor": 4.0, "original": 2048, "fast": 32.0, "slow": 1.0}
+    order = [{"type": "delta", "mixer": delta, "mlp": mlp},
+             {"type": "attention", "mixer": dict(base, rot={"base": 5e5, "dims": 64}), "mlp": mlp},
+             {"type": "attention_2", "mixer": dict(base, rot={"base": 5e5, "dims": 64, "scaling": scaling}), "mlp": mlp}]
+    ronolorn = {"architecture": "Ronolorn", "vocab": vocab, "width": width, "streams": 4, "norm": {"eps": 1e-6},
+                "embedding": {"scale": 12.0}, "layers": order + order}
+    return ronolorn, dudatar
 
 
 def _time_us(fn, iters=20):
@@ -1091,17 +1115,161 @@ def gunulorn_kernel_table(width, peaks):
     return out
 
 
+def ronolorn_kernel_table(width, peaks):
+    """Ronolorn's kernels beside the like kernels of Dudatar, Tarivik, Delilorn and Gunulorn at this width, time over
+    roofline time.  The memory (convolution, delta rule, norm and gate) and the delta rule alone beside Dudatar's gated scan
+    and Tarivik's state space (roofline: the slower of bytes over the copy bandwidth and 32-bit multiply-adds over the
+    CUDA cores' rate, three per state element and token for the delta rule, which reads the state twice, two for a scan);
+    window attention with and without one more in the softmax sum beside Delilorn's window with kept tokens (prefill:
+    FLOPs of the visible keys; decode: bytes of the cached keys and values); joint norm, rotation and cache write of tied
+    values, and rotation and cache write, beside Delilorn's rotation and cache write; what lies between two sub-layers on four
+    streams beside Dudatar's add + layer norm; the feed-forward beside Dudatar's; the activation alone beside the gated
+    one (bytes).  All launches are replayed from a graph: the host's time between them is not in the figures."""
+    import torch
+    from tinyserve_b200.engine.batch import GroupView, StepContext
+    from tinyserve_b200.kernels import ops
+    from tinyserve_b200.parts.mlp import PlainMLP
+    from tinyserve_b200.parts.rotary import Rotary
+    dev, bf = "cuda:0", torch.bfloat16
+    raw, beside = ronolorn_shapes(width)
+    mem, win, ff, S = raw["layers"][0]["mixer"], raw["layers"][1]["mixer"], raw["layers"][0]["mlp"]["ff"], raw["streams"]
+    gla, ffd = beside["layers"][0]["mixer"], beside["layers"][0]["mlp"]["ff"]
+    ssm = tarivik_shapes(width)[0]["layers"][0]["mixer"]["right"]
+    H, G, D = win["heads"], win["kv_heads"], 128
+    fma_tflops = ops.num_sms() * 128 * 2 * 1.965e9 / 1e12
+    out = {}
+    rnd = lambda *s, scale=1.0: (torch.randn(*s, device=dev) * scale).to(bf)
+
+    def frac(key, us, roof):
+        out[key] = {"us": round(us, 1), "roofline_us": round(roof, 2), "frac": round(roof / us, 3)}
+
+    def rotary(dims, interleaved):
+        cos, sin = Rotary.tables(dims, 5e5, CONTEXT)
+        return type("R", (), {"cos": cos.to(dev), "sin": sin.to(dev), "rotary_dim": dims, "interleaved": interleaved})()
+
+    for name, lengths, starts in (("prefill_2048", [2048], [0]), ("decode_b8", [1] * 8, [2048] * 8)):
+        T, B = sum(lengths), len(lengths)
+        timed = _time_graph_us
+        moved = lambda bytes_: bytes_ / (peaks["hbm_gbs"] * 1e3)
+        kv_len, page = starts[0] + lengths[0], 64
+        pages_per = -(-kv_len // page)
+        cu = torch.tensor([0] + list(torch.tensor(lengths).cumsum(0)), dtype=torch.int32, device=dev)
+        table = (torch.arange(B * pages_per, dtype=torch.int32, device=dev) + 1).view(B, pages_per)
+        positions = torch.cat([torch.arange(s, s + m) for s, m in zip(starts, lengths)]).int().to(dev)
+        slots = torch.cat([table[b, (s + torch.arange(m, device=dev)) // page] * page + (s + torch.arange(m, device=dev)) % page
+                           for b, (s, m) in enumerate(zip(starts, lengths))]).int()
+        kc, vc = (torch.randn(B * pages_per + 1, G, page, D, device=dev).to(bf) for _ in range(2))
+        sc = StepContext()
+        sc.num_tokens, sc.num_requests, sc.max_q_len, sc.max_kv_len = T, B, max(lengths), kv_len
+        sc.cu_q, sc.kv_lens, sc.positions = cu, torch.full((B,), kv_len, dtype=torch.int32, device=dev), positions
+        sc.state_slots, sc.fresh = torch.arange(B, dtype=torch.int32, device=dev), torch.zeros(B, dtype=torch.int32, device=dev)
+        sc.host = {"cu_q": cu.tolist(), "kv_lens": [kv_len] * B}
+        view = GroupView(page, pages_per, None, table, kc.shape[0])
+        # the memory
+        Hm, Gm, n, nv, taps = mem["heads"], mem["kv_heads"], mem["dim"], mem["vdim"], mem["conv"]
+        qk, C = Gm * n, 2 * Gm * n + Hm * nv
+        proj, logits, cw = rnd(T, C + Hm * nv), torch.randn(T, 2 * Hm, device=dev), rnd(C, taps, scale=0.5)
+        state, conv_state = torch.zeros(B, Hm, n, nv, device=dev), torch.zeros(B, taps - 1, C, device=dev)
+        bias, rate, wn = torch.zeros(Hm, device=dev), torch.full((Hm,), -3.0, device=dev), torch.ones(nv, device=dev, dtype=bf)
+
+        def delta(x):
+            return ops.delta_rule(x[:, :qk], x[:, qk:2 * qk], x[:, 2 * qk:C], proj[:, C:], logits, bias, rate, state, sc, Hm, n, nv, wn, 1e-6, bf,
+                                  q_scale=n ** -0.5, qk_group=Hm // Gm)
+        convolved = lambda: ops.causal_conv(proj[:, :C], cw, conv_state, sc, bf, activation="silu")
+        xc = convolved()
+
+        def recurrence(heads, n_, nv_, row_bytes, per_element):
+            return max(moved(T * row_bytes + 2 * B * heads * n_ * nv_ * 4), per_element * T * heads * n_ * nv_ / (fma_tflops * 1e6))
+        rows = (C + 2 * Hm * nv) * 2 + 2 * Hm * 4
+        frac(f"delta_rule_{name}", timed(lambda: delta(xc)), recurrence(Hm, n, nv, rows, 6.0))
+        frac(f"convolution_delta_rule_{name}", timed(lambda: delta(convolved())), recurrence(Hm, n, nv, rows, 6.0))
+        frac(f"convolution_{name}", timed(convolved), moved(T * C * 4))
+        Hg, ng, nvg = gla["heads"], gla["dim"], gla["vdim"]
+        pg, z, sg = rnd(T, 2 * Hg * ng + 2 * Hg * nvg), torch.randn(T, Hg * ng, device=dev) + 3, torch.zeros(B, Hg, ng, nvg, device=dev)
+        wg = torch.ones(nvg, device=dev, dtype=bf)
+        frac(f"dudatar_gated_scan_{name}", timed(lambda: ops.linear_attention(
+            pg[:, :Hg * ng], pg[:, Hg * ng:2 * Hg * ng], pg[:, 2 * Hg * ng:2 * Hg * ng + Hg * nvg], pg[:, 2 * Hg * ng + Hg * nvg:], sg, sc, Hg, ng, nvg,
+            bf, decay_logits=z, tau=8.0, q_scale=ng ** -0.5, norm_weight=wg, eps=1e-5)),
+            recurrence(Hg, ng, nvg, (2 * Hg * ng + 3 * Hg * nvg) * 2 + Hg * ng * 4, 4.0))
+        Hs, nvs, ns, groups = ssm["heads"], ssm["vdim"], ssm["state"], ssm["groups"]
+        inner, Cs = Hs * nvs, Hs * nvs + 2 * groups * ns
+        ps, dt_raw, ss = rnd(T, inner + Cs), torch.randn(T, Hs, device=dev), torch.zeros(B, Hs, ns, nvs, device=dev)
+        cws, css = rnd(Cs, ssm["conv"], scale=0.3), torch.zeros(B, ssm["conv"] - 1, Cs, device=dev)
+        hs, ws = torch.zeros(Hs, device=dev), torch.ones(inner, device=dev)
+
+        def state_space():
+            x = ops.causal_conv(ps[:, inner:], cws, css, sc, bf, activation="silu")
+            o = ops.linear_attention(x[:, inner + groups * ns:], x[:, inner:inner + groups * ns], x[:, :inner], None, ss, sc, Hs, ns, nvs, bf,
+                                     step_sizes=(dt_raw, hs, hs), qk_group=Hs // groups, raw=True)
+            return ops.ssm_finish(o, x[:, :inner], hs, ps[:, :inner], ws, 1, 1e-6, Hs, nvs, bf)
+        frac(f"tarivik_state_space_{name}", timed(state_space), recurrence(Hs, ns, nvs, (Cs + 2 * inner) * 2 + Hs * 4, 4.0))
+        # attention
+        q = rnd(T, H, D)
+
+        def attention(**kw):
+            run = lambda: ops.paged_attention(q, kc, vc, view, sc, D ** -0.5, **kw)
+            run()                                                                     # (work lists)
+            return timed(run)
+
+        def roof(window, keep=0):
+            pos = torch.arange(kv_len - lengths[0], kv_len)
+            seen = torch.minimum(pos + 1, torch.full_like(pos, window)) + torch.clamp(
+                torch.minimum(pos + 1 - window, torch.full_like(pos, keep)), min=0)
+            seen = float(seen.sum())
+            return 4.0 * H * D * seen / (peaks["bf16_tflops"] * 1e6) if T > B else moved(B * seen * 2 * G * D * 2)
+        size = win["mask"]["size"]
+        frac(f"window_attention_{name}", attention(window=size), roof(size))
+        frac(f"window_attention_one_more_{name}", attention(window=size, sinks=torch.zeros(H, device=dev)), roof(size))
+        frac(f"delilorn_window_attention_{name}", attention(window=size, keep_first=4), roof(size, 4))
+        qkv = rnd(T, (H + 2 * G) * D)
+        qw, kw_ = torch.ones(H * D, device=dev, dtype=bf), torch.ones(G * D, device=dev, dtype=bf)
+        q_end, k_end = H * D, (H + G) * D
+        pairs, halves = rotary(64, True), rotary(64, False)
+        kwargs = dict(k_cache=kc, v_cache=vc, slot_mapping=slots, page_size=page)
+        tied = rnd(T, (H + G) * D)
+        frac(f"joint_norm_rotary_tied_cache_write_{name}", timed(lambda: ops.joint_norm_kvwrite(
+            tied[:, :q_end], tied[:, q_end:], tied[:, q_end:], H, G, D, D, D, qw, kw_, 1e-6, rotary=pairs, positions=positions, **kwargs)),
+            moved(T * ((H + G) + (H + 2 * G)) * D * 2))
+        rope = lambda rot: ops.rope_unit_kvwrite(qkv[:, :q_end], qkv[:, q_end:k_end], qkv[:, k_end:], positions, H, G, D, D, D, rotary=rot, **kwargs)
+        frac(f"rotary_cache_write_{name}", timed(lambda: rope(pairs)), moved(T * (H + 2 * G) * D * 4))
+        frac(f"delilorn_rotary_cache_write_{name}", timed(lambda: rope(halves)), moved(T * (H + 2 * G) * D * 4))
+        # between two sub-layers
+        streams = ops.Streams(torch.randn(T, width, device=dev), S)
+        streams.data = torch.randn(T, S, width, device=dev)
+        y, y2, res = rnd(T, width), rnd(T, width), torch.randn(T, width, device=dev)
+        mix, vec, w1 = (torch.eye(S, device=dev) + 0.01).to(bf), torch.full((S,), 0.5, device=dev, dtype=bf), torch.ones(width, device=dev, dtype=bf)
+        frac(f"streams_{S}_mix_layernorm_{name}", timed(lambda: ops.stream_norm(ops.StreamMix(y, mix, vec), streams, vec, w1, 1e-6, bf)),
+             moved(T * width * (8 * S + 4)))
+        frac(f"dudatar_add_layernorm_{name}", timed(lambda: ops.add_layernorm(ops.PairSum(y, y2), res, w1, 1e-6, bf)), moved(T * width * (8 + 4 + 2)))
+        # feed-forward
+        h, part = rnd(T, width), PlainMLP(width, ff)
+        part.bind({"up_proj.weight": rnd(ff, width, scale=0.02), "down_proj.weight": rnd(width, ff, scale=0.02)})
+        gate_up, gdown = rnd(2 * ffd, width, scale=0.02), rnd(width, ffd, scale=0.02)
+        block = ops.GATED_BLOCK if ffd % ops.GATED_BLOCK == 0 else 0
+        us = timed(lambda: ops.materialize(part.forward(h, None)))
+        us_gated = timed(lambda: ops.materialize(ops.linear(ops.gated_linear(h, gate_up, "gelu_tanh", block), gdown)))
+        flops = lambda f: f / (peaks["bf16_tflops"] * 1e6)
+        frac(f"feed_forward_{name}", us, flops(4.0 * T * width * ff) if T > B else moved(2.0 * width * ff * 2))
+        frac(f"dudatar_feed_forward_{name}", us_gated, flops(6.0 * T * width * ffd) if T > B else moved(3.0 * width * ffd * 2))
+        if T > B:
+            z1, z2 = rnd(T, ff), rnd(T, 2 * ffd)
+            frac(f"relu_squared_{name}", timed(lambda: ops.plain_activation_(z1, "relu_squared")), moved(T * ff * 4))
+            frac(f"dudatar_gated_activation_{name}", timed(lambda: ops.gated_activation(z2, "gelu_tanh", block)), moved(T * ffd * 6))
+    return out
+
+
 # design -> (its shapes and those of the model beside it, its kernel table, the name of the model beside it)
 ARCH_BENCHES = {"dudatar": (dudatar_shapes, kernel_table, "qwen3"), "delilorn": (delilorn_shapes, delilorn_kernel_table, "qwen3"),
                 "tarivik": (tarivik_shapes, tarivik_kernel_table, "delilorn"),
                 "babadra": (babadra_shapes, babadra_kernel_table, "delilorn"),
-                "gunulorn": (gunulorn_shapes, gunulorn_kernel_table, "babadra")}
+                "gunulorn": (gunulorn_shapes, gunulorn_kernel_table, "babadra"),
+                "ronolorn": (ronolorn_shapes, ronolorn_kernel_table, "dudatar")}
 
 
 def arch_main(a) -> int:
     """``--arch dudatar`` / ``--arch delilorn``: the design beside Qwen3 at equal size; ``--arch tarivik`` and
     ``--arch babadra``: beside Delilorn, the closest design (experts, latent attention, matrix-state mixers);
-    ``--arch gunulorn``: beside Babadra.  One JSON line."""
+    ``--arch gunulorn``: beside Babadra; ``--arch ronolorn``: beside Dudatar.  One JSON line."""
     import torch
     from tinyserve_b200 import LLM
     from tinyserve_b200.config import config_from_dict
@@ -1171,10 +1339,10 @@ def main() -> int:
     ap.add_argument("--no-points", action="store_true", help="skip batch 1 / 64 and prefill")
     ap.add_argument("--no-workloads", action="store_true",
                     help="skip the 0.6B burst, the 32B run and the long-context decode")
-    ap.add_argument("--arch", choices=["qwen3", "dudatar", "delilorn", "tarivik", "babadra", "gunulorn"], default="qwen3",
+    ap.add_argument("--arch", choices=["qwen3", "dudatar", "delilorn", "tarivik", "babadra", "gunulorn", "ronolorn"], default="qwen3",
                     help="dudatar, delilorn: measure that design beside Qwen3 at equal size instead of the default workload; "
-                         "tarivik, babadra: beside Delilorn; gunulorn: beside Babadra")
-    ap.add_argument("--sizes", default="2048,4096", help="--arch dudatar / delilorn / tarivik / babadra / gunulorn: model widths to measure")
+                         "tarivik, babadra: beside Delilorn; gunulorn: beside Babadra; ronolorn: beside Dudatar")
+    ap.add_argument("--sizes", default="2048,4096", help="--arch dudatar / delilorn / tarivik / babadra / gunulorn / ronolorn: model widths to measure")
     a = ap.parse_args()
     if a.impl == "reference":
         return reference_main(a)

@@ -157,7 +157,7 @@ def _plain_memory(q, k, v, gate, logits, bias, rate, norm, eps, H, G, n, nv, sta
 
 @pytest.mark.parametrize("dtype,tol", [(torch.float32, 2e-5), (torch.bfloat16, 8e-3)])
 @pytest.mark.parametrize("H,G,n,nv", [(4, 2, 20, 12), (3, 3, 12, 40), (6, 2, 36, 10), (4, 1, 32, 48), (2, 2, 64, 80), (2, 1, 128, 128),
-                                      (1, 1, 256, 300), (5, 1, 8, 1), (2, 2, 48, 33), (3, 1, 96, 64)])
+                                      (1, 1, 256, 300), (1, 1, 512, 18), (5, 1, 8, 1), (2, 2, 48, 33), (3, 1, 96, 64)])
 @pytest.mark.parametrize("tile", [None, 0, 1, 16, 40])
 def test_memory_under_the_delta_rule(dtype, tol, H, G, n, nv, tile):
     """Portions of every size (one token, shorter and longer than the staged chunk), requests beside one

@@ -2372,9 +2372,11 @@ def stream_norm(x, streams, read, weight, eps, out_dtype, bias=None, centred=Tru
 # ----------------------------------------------------------------------------- gated delta rule
 DELTA_MAX_KEY_DIM = 1024
 #: requests of up to this many tokens in a step run the wide form of the kernel (the state's transfer counts), longer
-#: portions the narrow one in tiles of DELTA_TILE value columns (the chain from token to token counts)
-DELTA_WIDE_MAX_TOKENS = 4
-DELTA_TILE = 16
+#: portions the narrow one (the chain from token to token counts), in blocks of DELTA_TILES value columns: the first where
+#: they then fit the SMs at once, else the second (measured on B200, one prompt of 2,048 tokens, heads of 128 x 128: 16
+#: heads 287 us against 394, 32 heads 566 us against 413)
+DELTA_WIDE_MAX_TOKENS = 8
+DELTA_TILES = (16, 32)
 
 
 def delta_rule(q, k, v, gate, logits, bias, rate, state, ctx, num_heads, key_dim, value_dim, norm_weight, eps, out_dtype,
@@ -2398,15 +2400,19 @@ def delta_rule(q, k, v, gate, logits, bias, rate, state, ctx, num_heads, key_dim
         raise ValueError(f"delta_rule: key sizes of up to {DELTA_MAX_KEY_DIM}")
     longest = max(1, min(getattr(ctx, "max_q_len", 0) or T, T))
     if tile is None:
-        tile = 0 if longest <= DELTA_WIDE_MAX_TOKENS else DELTA_TILE
+        blocks = ctx.num_requests * H * -(-value_dim // DELTA_TILES[0])
+        tile = 0 if longest <= DELTA_WIDE_MAX_TOKENS else DELTA_TILES[0 if blocks <= num_sms() else 1]
     lib = build.load_unit("delta_rule.cu", {"TS_KEY_DIM": key_dim})
     spread = lib.ts_delta_rule_column_tiles(c_int(value_dim), c_int(tile)) > 1
+    lib.ts_delta_rule_scratch.restype = c_longlong
     raw = torch.empty(T, H * value_dim, dtype=torch.float32, device=q.device) if spread else None
+    groups = torch.empty(lib.ts_delta_rule_scratch(c_int(T), c_int(ctx.num_requests), c_int(H)), dtype=torch.float32,
+                         device=q.device) if tile > 0 else None
     out = torch.empty(T, H * value_dim, dtype=out_dtype, device=q.device)
     _check(lib, lib.ts_delta_rule(
         c_int(_dt(q)), *_columns(q), *_columns(k), *_columns(v), *_columns(gate), _ptr(logits), c_longlong(logits.stride(0)), _ptr(bias),
         c_int(_f32(bias)), _ptr(rate), c_int(_f32(rate)), c_float(q_scale), _ptr(state), _ptr(ctx.state_slots), _ptr(ctx.fresh),
         _ptr(ctx.cu_q), c_int(ctx.num_requests), c_int(longest), c_int(T), _ptr(norm_weight), c_int(_f32(norm_weight)), c_float(eps),
-        _ptr(out), c_longlong(out.stride(0)), _ptr(raw), c_int(H), c_int(value_dim), c_int(qk_group), c_int(tile), _stream()),
-        2 if spread else 1)
+        _ptr(out), c_longlong(out.stride(0)), _ptr(raw), c_int(H), c_int(value_dim), c_int(qk_group), c_int(tile), _ptr(groups), _stream()),
+        1 + int(spread) + int(tile > 0))
     return out
