@@ -476,12 +476,12 @@ def ronolorn_shapes(width):
     mlp = {"kind": "dense", "ff": dudatar["layers"][0]["mlp"]["ff"] * 3 // 2}
     base = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 1024}}
     delta = {"heads": heads, "kv_heads": heads // 2, "dim": 128, "vdim": 128, "conv": 4}
-    scaling = {"factor": 4.0, "original": 2048, "fast": 32.0, "slow": 1.0}
+    scaling = {"factor": 8.0, "original": 1024, "fast": 16.0, "slow": 1.0}
     order = [{"type": "delta", "mixer": delta, "mlp": mlp},
-             {"type": "attention", "mixer": dict(base, rot={"base": 5e5, "dims": 64}), "mlp": mlp},
-             {"type": "attention_2", "mixer": dict(base, rot={"base": 5e5, "dims": 64, "scaling": scaling}), "mlp": mlp}]
+             {"type": "attention", "mixer": dict(base, rot={"base": 1e6, "dims": 64}), "mlp": mlp},
+             {"type": "attention_2", "mixer": dict(base, rot={"base": 1e6, "dims": 64, "scaling": scaling}), "mlp": mlp}]
     ronolorn = {"architecture": "Ronolorn", "vocab": vocab, "width": width, "streams": 4, "norm": {"eps": 1e-6},
-                "embedding": {"scale": 12.0}, "layers": order + order}
+                "embedding": {"scale": float(width) ** 0.5}, "layers": order + order}
     return ronolorn, dudatar
 
 
